@@ -73,7 +73,7 @@ __device__ __forceinline__ float gelu_erf(float x) {
   return 0.5f * x * (1.f + erff(x * 0.7071067811865476f));
 }
 
-enum Activation : int { ACT_NONE = 0, ACT_GELU_TANH = 1, ACT_GELU_ERF = 2 };
+enum Activation : int { ACT_NONE = 0, ACT_GELU_TANH = 1, ACT_GELU_ERF = 2, ACT_RELU_SQUARED = 3 };
 
 // The tanh form with the hardware's approximate tanh (one special-function instruction,
 // relative error about 2^-11): for results that are rounded to bfloat16 (2^-8) right after.
@@ -84,9 +84,15 @@ __device__ __forceinline__ float gelu_tanh_fast(float x) {
   return 0.5f * x * (1.f + t);
 }
 
+__device__ __forceinline__ float relu_squared(float x) {
+  const float y = fmaxf(x, 0.f);
+  return y * y;
+}
+
 __device__ __forceinline__ float activate(float x, int act) {
   if (act == ACT_GELU_TANH) return gelu_tanh(x);
   if (act == ACT_GELU_ERF) return gelu_erf(x);
+  if (act == ACT_RELU_SQUARED) return relu_squared(x);
   return x;
 }
 
@@ -94,6 +100,7 @@ __device__ __forceinline__ float activate(float x, int act) {
 __device__ __forceinline__ float activate_to_bf16(float x, int act) {
   if (act == ACT_GELU_TANH) return gelu_tanh_fast(x);
   if (act == ACT_GELU_ERF) return gelu_erf(x);
+  if (act == ACT_RELU_SQUARED) return relu_squared(x);
   return x;
 }
 

@@ -9,8 +9,9 @@
 // column 0 (H * dim), keys at k_off (G * dim), values at v_off (G * vdim): with norm weights
 // the whole query projection and the whole key projection are each divided by their root mean
 // square (one mean over all heads' entries, eps inside the root) and multiplied by a weight
-// per entry; queries go to `q` in the compute type, the key and value into the row's cache
-// slot (pages [page][kv head][slot][dim or vdim]).
+// per entry; with rotation frequencies the first rot_dims entries of every query and key head
+// are then rotated by the row's position; queries go to `q` in the compute type, the key and
+// value into the row's cache slot (pages [page][kv head][slot][dim or vdim]).
 //
 // attention: scores scale * (q . k), softmax and the weighted sum in fp32, the result times
 // sigmoid(gate) entry by entry when a gate (fp32, [row][H * vdim]) is given. The visible keys
@@ -22,6 +23,7 @@
 // down). Prompt portions in bfloat16 run on the tensor cores in attention_prefill.cu, which
 // takes the same mask, value size and gate.
 #include "common.cuh"
+#include "rope.cuh"
 
 namespace ayk {
 
@@ -34,10 +36,16 @@ gated_prepare_kernel(const float* __restrict__ proj, int ld_proj, int k_off, int
                      const float* __restrict__ q_weight, const float* __restrict__ k_weight,
                      float eps, const int* __restrict__ slots, T* __restrict__ k_pages,
                      T* __restrict__ v_pages, int page_size, T* __restrict__ q, int ld_q, int H,
-                     int G, int dim, int vdim) {
+                     int G, int dim, int vdim, const int* __restrict__ positions,
+                     const double* __restrict__ freq, int rot_dims, int rot_layout) {
   __shared__ float scratch[33];
+  __shared__ float cos_s[ROPE_MAX_PAIRS], sin_s[ROPE_MAX_PAIRS];
   pdl_launch_dependents();
   const int row = blockIdx.x, tid = threadIdx.x;
+  if (rot_dims > 0) {
+    rope_fill_table_reduced(cos_s, sin_s, positions[row], freq, rot_dims / 2);
+    __syncthreads();
+  }
   const int qn = H * dim, kn = G * dim, vn = G * vdim;
   const int slot = (slots != nullptr && k_pages != nullptr) ? slots[row] : -1;
   pdl_wait_for(proj);
@@ -53,16 +61,27 @@ gated_prepare_kernel(const float* __restrict__ proj, int ld_proj, int k_off, int
     for (int i = tid; i < kn; i += blockDim.x) s += src[k_off + i] * src[k_off + i];
     k_inv = 1.f / sqrtf(block_sum(s, scratch) / (float)kn + eps);
   }
+  // entry i of a projection (entry d of its head), normed and rotated
+  auto entry = [&](const float* x, const float* w, float inv, int i, int d) {
+    const float v = x[i] * inv * (w != nullptr ? w[i] : 1.f);
+    if (d >= rot_dims) return v;
+    const bool halves = rot_layout == ROPE_HALVES;
+    const int half = rot_dims / 2, pair = halves ? d % half : d >> 1;
+    const bool second = halves ? d >= half : (d & 1);
+    const int apart = halves ? half : 1, j = second ? i - apart : i + apart;
+    const float o = x[j] * inv * (w != nullptr ? w[j] : 1.f);
+    return second ? v * cos_s[pair] + o * sin_s[pair] : v * cos_s[pair] - o * sin_s[pair];
+  };
   T* q_row = q + (size_t)row * ld_q;
   for (int i = tid; i < qn; i += blockDim.x) {
-    stf(q_row + i, src[i] * q_inv * (q_weight != nullptr ? q_weight[i] : 1.f));
+    stf(q_row + i, entry(src, q_weight, q_inv, i, i % dim));
   }
   if (slot < 0) return;
   const size_t page = slot / page_size, at = slot % page_size;
   for (int i = tid; i < kn; i += blockDim.x) {
     const int g = i / dim, d = i % dim;
     stf(k_pages + ((page * G + g) * page_size + at) * dim + d,
-        src[k_off + i] * k_inv * (k_weight != nullptr ? k_weight[i] : 1.f));
+        entry(src + k_off, k_weight, k_inv, i, d));
   }
   for (int i = tid; i < vn; i += blockDim.x) {
     const int g = i / vdim, d = i % vdim;
@@ -398,14 +417,19 @@ int gated_attention(const void* q, int ld_q, const void* k_pages, const void* v_
 AYK_API void ayk_set_pdl(int on) { ayk::pdl_enabled() = on; }
 
 // type: 0 = float32, 1 = bfloat16 (of q and the pages). Norm weights, slots and pages may be
-// null (no norm; nothing stored).
+// null (no norm; nothing stored). rot_dims 0: no rotation (positions and freq may be null).
 AYK_API int ayk_gated_prepare(const float* proj, int ld_proj, int k_off, int v_off,
                               const float* q_weight, const float* k_weight, float eps,
                               const int* slots, void* k_pages, void* v_pages, int page_size,
                               void* q, int ld_q, int rows, int heads, int kv_heads, int dim,
-                              int vdim, int type, void* stream) {
+                              int vdim, const int* positions, const double* freq, int rot_dims,
+                              int rot_layout, int type, void* stream) {
   using namespace ayk;
   if (rows == 0) return AYK_OK;
+  if (rot_dims < 0 || rot_dims % 2 || rot_dims > dim || rot_dims > 2 * ROPE_MAX_PAIRS ||
+      (rot_dims > 0 && (positions == nullptr || freq == nullptr))) {
+    return AYK_BAD_ARGUMENT;
+  }
   if (rows < 0 || heads < 1 || kv_heads < 1 || heads % kv_heads || dim < 1 || vdim < 1 ||
       proj == nullptr || q == nullptr || ld_q < heads * dim || k_off < heads * dim ||
       v_off < k_off + kv_heads * dim || ld_proj < v_off + kv_heads * vdim ||
@@ -417,13 +441,15 @@ AYK_API int ayk_gated_prepare(const float* proj, int ld_proj, int k_off, int v_o
   if (type == 0) {
     return launch_kernel(gated_prepare_kernel<float>, dim3(rows), dim3(256), 0, s, 1, proj,
                          ld_proj, k_off, v_off, q_weight, k_weight, eps, slots, (float*)k_pages,
-                         (float*)v_pages, page_size, (float*)q, ld_q, heads, kv_heads, dim, vdim);
+                         (float*)v_pages, page_size, (float*)q, ld_q, heads, kv_heads, dim, vdim,
+                         positions, freq, rot_dims, rot_layout);
   }
   if (type == 1) {
     return launch_kernel(gated_prepare_kernel<__nv_bfloat16>, dim3(rows), dim3(256), 0, s, 1,
                          proj, ld_proj, k_off, v_off, q_weight, k_weight, eps, slots,
                          (__nv_bfloat16*)k_pages, (__nv_bfloat16*)v_pages, page_size,
-                         (__nv_bfloat16*)q, ld_q, heads, kv_heads, dim, vdim);
+                         (__nv_bfloat16*)q, ld_q, heads, kv_heads, dim, vdim, positions, freq,
+                         rot_dims, rot_layout);
   }
   return AYK_BAD_ARGUMENT;
 }

@@ -86,7 +86,7 @@ int gemm_simt(const void* a, int lda, const void* w, int ldw, const float* bias,
               int ldo, int M, int N, int K, int act, cudaStream_t stream) {
   if (M == 0 || N == 0) return AYK_OK;
   if (M < 0 || N < 0 || K < 1 || lda < K || ldw < K || ldo < N) return AYK_BAD_ARGUMENT;
-  if (act < ACT_NONE || act > ACT_GELU_ERF) return AYK_BAD_ARGUMENT;
+  if (act < ACT_NONE || act > ACT_RELU_SQUARED) return AYK_BAD_ARGUMENT;
   const long long gy = (M + BM - 1) / BM;
   if (gy > 65535) return AYK_TOO_LARGE;
   dim3 grid((N + BN - 1) / BN, (unsigned)gy);

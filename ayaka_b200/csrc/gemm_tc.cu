@@ -1559,7 +1559,7 @@ AYK_API int ayk_gemm_bf16_tc(const void* a, int lda, const void* w, int ldw, con
   if (M < 0 || N < 0 || K < 1 || lda < K || ldw < K || ldo < N || status == nullptr) {
     return AYK_BAD_ARGUMENT;
   }
-  if (mode < OUT_BF16 || mode > OUT_RESIDUAL_F32 || act < ACT_NONE || act > ACT_GELU_ERF ||
+  if (mode < OUT_BF16 || mode > OUT_RESIDUAL_F32 || act < ACT_NONE || act > ACT_RELU_SQUARED ||
       (mode == OUT_RESIDUAL_F32 && act != ACT_NONE)) {
     return AYK_BAD_ARGUMENT;
   }

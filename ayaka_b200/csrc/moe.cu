@@ -11,7 +11,8 @@
 //            g = min(W_gate h, limit), u = clamp(W_up h, -limit, limit) and writes
 //            y = g sigmoid(alpha g) (u + shift); the second writes W_down y per pair in
 //            fp32 (limit = infinity, alpha = 1, shift = 0: silu(g) u);
-//   join:    dst[row] (+)= scale * sum_choice share * (W_down y)[pair], choices in order.
+//   join:    dst[row] (+)= scale * sum_choice share * (W_down y)[pair], choices in order; a
+//            choice at or beyond E is an identity expert, whose output is the row's input.
 // A pair's result does not depend on its place in a tile or on the other pairs: every output
 // element is one sum over k in a fixed order. Experts' matrices lie one under the other:
 // w_in [E][2 * ff][width] (an expert's gate rows, then its up rows), w_out [E][width][ff]. An
@@ -84,27 +85,45 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, int ld, int r
   for (int j = 32 + lane; j < top; j += 32) share[(size_t)row * top + j] /= total;
 }
 
-// Routing by scores with groups: s = sigmoid(logit); the experts form `groups` equal groups of
-// neighbours, a group's score is the sum of its two largest s (its only one when a group is one
-// expert), and only experts of the `keep` best groups can be chosen; of those the `top` largest
-// s are taken (ties to the smaller index, also among groups). share = factor * s, divided by
-// the chosen ones' sum when `renorm` is set. One warp per row; the row's scores, the groups'
-// scores and the kept groups' marks lie in the warp's part of shared memory.
+// Routing by scores with groups: s = sigmoid(logit), or the softmax over all experts with
+// `softmax`; what is compared is s + correction (when given). The experts form `groups` equal
+// groups of neighbours, a group's score is the sum of its two largest (its only one when a group
+// is one expert), and only experts of the `keep` best groups can be chosen; of those the `top`
+// largest are taken (ties to the smaller index, also among groups). share = factor * s (without
+// the correction), divided by the chosen ones' sum + `floor` when `renorm` is set. One warp per
+// row; the row's scores, what is compared, the groups' scores and the kept groups' marks lie in
+// the warp's part of shared memory.
 __global__ void moe_route_scored_kernel(const float* __restrict__ logits, int ld, int rows, int E,
                                         int top, int groups, int keep, float factor, int renorm,
-                                        int* __restrict__ chosen, float* __restrict__ share) {
+                                        int softmax, const float* __restrict__ correction,
+                                        float floor, int* __restrict__ chosen,
+                                        float* __restrict__ share) {
   extern __shared__ float route_smem[];
   pdl_launch_dependents();
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int row = blockIdx.x * (blockDim.x >> 5) + warp;
   if (row >= rows) return;
-  float* s = route_smem + (size_t)warp * (E + 2 * groups);
+  float* score = route_smem + (size_t)warp * (2 * E + 2 * groups);
+  float* s = score + E;  // what is compared
   float* gs = s + E;
   int* kept = reinterpret_cast<int*>(gs + groups);
   const int per = E / groups;
   pdl_wait_for(logits);
   const float* z = logits + (size_t)row * ld;
-  for (int e = lane; e < E; e += 32) s[e] = 1.f / (1.f + expf(-z[e]));
+  float most = 0.f, below = 1.f;
+  if (softmax) {
+    most = -INFINITY;
+    for (int e = lane; e < E; e += 32) most = fmaxf(most, z[e]);
+    most = warp_max(most);
+    float all = 0.f;
+    for (int e = lane; e < E; e += 32) all += expf(z[e] - most);
+    below = warp_sum(all);
+  }
+  for (int e = lane; e < E; e += 32) {
+    const float v = softmax ? expf(z[e] - most) / below : 1.f / (1.f + expf(-z[e]));
+    score[e] = v;
+    s[e] = correction != nullptr ? v + correction[e] : v;
+  }
   __syncwarp();
   // the largest entry of v[0 .. n) not yet taken (taken ones are -inf), ties to the smaller index
   auto arg_max = [&](const float* v, int n, float& best, int& at) {
@@ -163,16 +182,17 @@ __global__ void moe_route_scored_kernel(const float* __restrict__ logits, int ld
     float best;
     int at;
     arg_max(s, E, best, at);
-    total += best;
+    const float weight = score[at];
+    total += weight;
     if (lane == 0) {
       s[at] = -INFINITY;
       chosen[(size_t)row * top + j] = at;
-      share[(size_t)row * top + j] = best * factor;
+      share[(size_t)row * top + j] = weight * factor;
     }
     __syncwarp();
   }
   if (renorm) {
-    for (int j = lane; j < top; j += 32) share[(size_t)row * top + j] /= total;
+    for (int j = lane; j < top; j += 32) share[(size_t)row * top + j] /= total + floor;
   }
 }
 
@@ -476,18 +496,25 @@ moe_tile_kernel(const T* __restrict__ a, int lda, const T* __restrict__ weight,
   });
 }
 
-// dst[row][c] (+)= scale[c] * sum_j share[row * top + j] * pair_out[row * top + j][c]
+// dst[row][c] (+)= scale[c] * sum_j share[row * top + j] * pair_out[row * top + j][c]; a pair whose
+// choice is `experts` or more takes hidden[row][c] instead (an identity expert; `hidden` and
+// `chosen` are null when there is none).
+template <typename T>
 __global__ void moe_join_kernel(const float* __restrict__ pair_out, int ld, const float* __restrict__ share,
-                                int top, const float* __restrict__ scale,
-                                float* __restrict__ dst, int ld_dst, int width, int accumulate) {
+                                const int* __restrict__ chosen, const T* __restrict__ hidden,
+                                int ld_hidden, int experts, int top,
+                                const float* __restrict__ scale, float* __restrict__ dst,
+                                int ld_dst, int width, int accumulate) {
   pdl_launch_dependents();
   const int row = blockIdx.x;
-  pdl_wait_for(pair_out, share, dst);
+  pdl_wait_for(pair_out, share, chosen, hidden, dst);
   for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < width; c += gridDim.y * blockDim.x) {
     float sum = 0.f;
     for (int j = 0; j < top; ++j) {
       const size_t pair = (size_t)row * top + j;
-      sum = fmaf(share[pair], pair_out[pair * ld + c], sum);
+      const bool identity = hidden != nullptr && chosen[pair] >= experts;
+      sum = fmaf(share[pair],
+                 identity ? ldf(hidden + (size_t)row * ld_hidden + c) : pair_out[pair * ld + c], sum);
     }
     if (scale != nullptr) sum *= scale[c];
     float* to = dst + (size_t)row * ld_dst + c;
@@ -552,8 +579,9 @@ AYK_API int ayk_moe_route(const float* logits, int ld, int rows, int experts, in
 // Scores instead of a softmax: see moe_route_scored_kernel. `groups` divides `experts`,
 // 1 <= keep <= groups, and the kept groups hold at least `top` experts.
 AYK_API int ayk_moe_route_scored(const float* logits, int ld, int rows, int experts, int top,
-                                 int groups, int keep, float factor, int renorm, int* chosen,
-                                 float* share, void* stream) {
+                                 int groups, int keep, float factor, int renorm, int softmax,
+                                 const float* correction, float floor, int* chosen, float* share,
+                                 void* stream) {
   using namespace ayk;
   if (rows == 0) return AYK_OK;
   if (rows < 0 || experts < 1 || top < 1 || groups < 1 || experts % groups || keep < 1 ||
@@ -562,12 +590,12 @@ AYK_API int ayk_moe_route_scored(const float* logits, int ld, int rows, int expe
     return AYK_BAD_ARGUMENT;
   }
   if (experts > MOE_MAX_EXPERTS) return AYK_TOO_LARGE;
-  const int per_warp = experts + 2 * groups;
+  const int per_warp = 2 * experts + 2 * groups;
   const int warps = per_warp <= 1024 ? 4 : 1;
   return launch_kernel(moe_route_scored_kernel, dim3((rows + warps - 1) / warps),
                        dim3(32 * warps), (size_t)warps * per_warp * sizeof(float),
                        (cudaStream_t)stream, 1, logits, ld, rows, experts, top, groups, keep,
-                       factor, renorm, chosen, share);
+                       factor, renorm, softmax, correction, floor, chosen, share);
 }
 
 // Three launches: align, the two grouped products. `sorted` holds max_tiles * tile_rows ints,
@@ -614,9 +642,12 @@ AYK_API int ayk_moe_experts(const void* hidden, int ld_hidden, const void* w_in,
   return AYK_BAD_ARGUMENT;
 }
 
-AYK_API int ayk_moe_join(const float* pair_out, int ld, const float* share, int rows, int top,
-                         const float* scale, float* dst, int ld_dst, int width, int accumulate,
-                         void* stream) {
+// `hidden` (type: 0 = float32, 1 = bfloat16) with `chosen`: choices from `experts` on are identity
+// experts; both null: there is none.
+AYK_API int ayk_moe_join(const float* pair_out, int ld, const float* share, const int* chosen,
+                         const void* hidden, int ld_hidden, int experts, int type, int rows,
+                         int top, const float* scale, float* dst, int ld_dst, int width,
+                         int accumulate, void* stream) {
   using namespace ayk;
   if (rows == 0) return AYK_OK;
   if (rows < 0 || top < 1 || width < 1 || pair_out == nullptr || share == nullptr ||
@@ -624,7 +655,16 @@ AYK_API int ayk_moe_join(const float* pair_out, int ld, const float* share, int 
     return AYK_BAD_ARGUMENT;
   }
   const int threads = 256, tiles = min(8, (width + threads - 1) / threads);
-  return launch_kernel(moe_join_kernel, dim3(rows, tiles), dim3(threads), 0,
-                       (cudaStream_t)stream, 1, pair_out, ld, share, top, scale, dst, ld_dst,
-                       width, accumulate);
+  if ((hidden == nullptr) != (chosen == nullptr) || (hidden != nullptr && ld_hidden < width)) {
+    return AYK_BAD_ARGUMENT;
+  }
+  if (type == 1) {
+    return launch_kernel(moe_join_kernel<__nv_bfloat16>, dim3(rows, tiles), dim3(threads), 0,
+                         (cudaStream_t)stream, 1, pair_out, ld, share, chosen,
+                         (const __nv_bfloat16*)hidden, ld_hidden, experts, top, scale, dst, ld_dst,
+                         width, accumulate);
+  }
+  return launch_kernel(moe_join_kernel<float>, dim3(rows, tiles), dim3(threads), 0,
+                       (cudaStream_t)stream, 1, pair_out, ld, share, chosen, (const float*)hidden,
+                       ld_hidden, experts, top, scale, dst, ld_dst, width, accumulate);
 }

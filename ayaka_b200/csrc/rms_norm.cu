@@ -11,7 +11,7 @@
 //   GATE_SILU_AFTER: the normalised, weighted value is multiplied by silu(gate) (the output
 //     gate of a gated-linear-attention layer).
 // `weight_period` > 0: the weight has that many entries and repeats along the row (one weight
-// shared by every head).
+// shared by every head); a null weight is all ones.
 //
 // norm_sum: several fp32 rows of the same width, each normalised over the whole width with a
 // weight of its own, are averaged, multiplied element by element by an optional scale and
@@ -59,13 +59,67 @@ __global__ void rms_norm_kernel(const float* __restrict__ x, int ld_x,
       const float z = gt[c];
       v *= z * sigmoid_f(z);
     }
-    v = v * inv * (weight_offset + w[weight_period > 0 ? (w_first + c) % weight_period : c]);
+    v *= inv;
+    if (weight != nullptr) {
+      v *= weight_offset + w[weight_period > 0 ? (w_first + c) % weight_period : c];
+    }
     if (gate_mode == GATE_SIGMOID_AFTER) v *= sigmoid_f(gt[c]);
     if (gate_mode == GATE_SILU_AFTER) {
       const float z = gt[c];
       v *= z * sigmoid_f(z);
     }
     stf(dst + c, v);
+  }
+}
+
+// The same for rows in several groups of at most 32 RG entries (the norm of every head of a
+// recurrent layer): a warp per (row, group), whose entries stay in its registers.
+template <typename TOut, int RG>
+__global__ void __launch_bounds__(256)
+rms_norm_groups_kernel(const float* __restrict__ x, int ld_x, const float* __restrict__ weight,
+                       float weight_offset, float eps, int groups, int group_width,
+                       const float* __restrict__ gate, int ld_gate, int gate_mode,
+                       TOut* __restrict__ out, int ld_out, int weight_period) {
+  pdl_launch_dependents();
+  const int r = blockIdx.x, lane = threadIdx.x & 31;
+  const int g = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  if (g >= groups) return;
+  const int first = g * group_width;
+  float wv[RG], xs[RG], zs[RG];
+#pragma unroll
+  for (int i = 0; i < RG; ++i) {
+    const int c = lane + 32 * i;
+    wv[i] = 1.f;
+    if (c < group_width && weight != nullptr) {
+      wv[i] = weight_offset + weight[weight_period > 0 ? (first + c) % weight_period : first + c];
+    }
+  }
+  pdl_wait_for(x, gate);
+  const float* src = x + (size_t)r * ld_x + first;
+  const float* gt = gate != nullptr ? gate + (size_t)r * ld_gate + first : nullptr;
+#pragma unroll
+  for (int i = 0; i < RG; ++i) {
+    const int c = lane + 32 * i;
+    xs[i] = c < group_width ? src[c] : 0.f;
+    zs[i] = gt != nullptr && c < group_width ? gt[c] : 0.f;
+  }
+  float s = 0.f;
+#pragma unroll
+  for (int i = 0; i < RG; ++i) {
+    if (gate_mode == GATE_SILU_BEFORE) xs[i] *= zs[i] * sigmoid_f(zs[i]);
+    s += xs[i] * xs[i];
+  }
+  const float inv = 1.f / sqrtf(warp_sum(s) / (float)group_width + eps);
+  TOut* dst = out + (size_t)r * ld_out + first;
+#pragma unroll
+  for (int i = 0; i < RG; ++i) {
+    const int c = lane + 32 * i;
+    if (c < group_width) {
+      float v = xs[i] * inv * wv[i];
+      if (gate_mode == GATE_SIGMOID_AFTER) v *= sigmoid_f(zs[i]);
+      if (gate_mode == GATE_SILU_AFTER) v *= zs[i] * sigmoid_f(zs[i]);
+      stf(dst + c, v);
+    }
   }
 }
 
@@ -89,12 +143,24 @@ int rms_norm(const float* x, int ld_x, const int* rows, const float* weight, flo
              int ld_out, int n, int width, int weight_period, cudaStream_t stream) {
   if (n == 0) return AYK_OK;
   if (n < 0 || width < 1 || groups < 1 || width % groups || ld_x < width || ld_out < width ||
-      !(eps > 0.f) || weight == nullptr || gate_mode < GATE_NONE ||
+      !(eps > 0.f) || gate_mode < GATE_NONE ||
       gate_mode > GATE_SILU_AFTER || ((gate_mode != GATE_NONE) != (gate != nullptr)) ||
       (gate != nullptr && ld_gate < width) || weight_period < 0) {
     return AYK_BAD_ARGUMENT;
   }
   const int group_width = width / groups;
+  if (groups > 1 && group_width <= 256 && rows == nullptr) {
+    const int warps = groups < 8 ? groups : 8;
+    const dim3 grid(n, (groups + warps - 1) / warps);
+#define AYK_NORM_GROUPS(RG)                                                                       \
+  return launch_kernel(rms_norm_groups_kernel<TOut, RG>, grid, dim3(32 * warps), 0, stream, 1, x, \
+                       ld_x, weight, weight_offset, eps, groups, group_width, gate, ld_gate,      \
+                       gate_mode, (TOut*)out, ld_out, weight_period)
+    if (group_width <= 64) AYK_NORM_GROUPS(2);
+    if (group_width <= 128) AYK_NORM_GROUPS(4);
+    AYK_NORM_GROUPS(8);
+#undef AYK_NORM_GROUPS
+  }
   const int threads = group_width >= 2048 ? 512 : (group_width >= 512 ? 256 : 128);
   return launch_kernel(rms_norm_kernel<TOut>, dim3(n, groups), dim3(threads), 0, stream, 1, x,
                        ld_x, rows, weight, weight_offset, eps, group_width, gate, ld_gate,

@@ -11,7 +11,8 @@ from __future__ import annotations
 import contextlib
 import math
 from collections.abc import Iterator
-from ctypes import c_float, c_int, c_longlong, c_void_p
+from dataclasses import dataclass
+from ctypes import Structure, byref, c_float, c_int, c_longlong, c_void_p, sizeof
 
 import torch
 
@@ -26,6 +27,7 @@ __all__ = [
     "attention_prefill",
     "cast_rows",
     "causal_conv_silu",
+    "conv_ring",
     "decode_splits",
     "delta_scan",
     "embed_rows",
@@ -34,6 +36,7 @@ __all__ = [
     "gated_decode",
     "gated_decode_shares",
     "gated_unit",
+    "LinearShape",
     "head_linear",
     "kv_store",
     "latent_attention",
@@ -44,6 +47,10 @@ __all__ = [
     "gla_scan",
     "layer_norm",
     "linear",
+    "linear_attention_chunks",
+    "linear_attention_decode",
+    "linear_chunk_floats",
+    "linear_chunks",
     "linear_normed",
     "logits_adjust",
     "logits_scale_cap",
@@ -77,7 +84,7 @@ __all__ = [
     "unary_rows",
 ]
 
-ACTIVATIONS = {"none": 0, "gelu_tanh": 1, "gelu_erf": 2}
+ACTIVATIONS = {"none": 0, "gelu_tanh": 1, "gelu_erf": 2, "relu_squared": 3}
 _TYPE = {torch.float32: 0, torch.bfloat16: 1}
 
 #: Which bfloat16 matrix-product kernel :func:`linear` launches: ``"tcgen05"`` (the tensor
@@ -123,7 +130,8 @@ _TIMED = ("embed_rows", "layer_norm", "linear", "linear_kv", "kv_store", "attent
           "mlstm_scan", "gla_scan", "talking_prepare", "talking_attention", "norm_sum",
           "moe_route", "moe_experts", "moe_join", "moe_route_scored", "cast_rows", "gated_unit",
           "norm_add", "gated_attention_prepare", "gated_attention", "gated_decode",
-          "unary_rows", "delta_scan", "pooled_prepare", "pooled_blocks", "pooled_attention")
+          "unary_rows", "delta_scan", "pooled_prepare", "pooled_blocks", "pooled_attention",
+          "conv_ring", "linear_attention_chunks", "linear_attention_decode")
 
 
 @contextlib.contextmanager
@@ -777,7 +785,7 @@ GATES = {"none": 0, "silu_before": 1, "sigmoid_after": 2, "silu_after": 3}
 ROPE_LAYOUTS = {"neighbours": 0, "halves": 1}
 
 
-def rms_norm(x: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor, *,
+def rms_norm(x: torch.Tensor, weight: torch.Tensor | None, eps: float, out: torch.Tensor, *,
              weight_offset: float = 0.0, groups: int = 1, rows: torch.Tensor | None = None,
              count: int | None = None, gate: torch.Tensor | None = None,
              gate_mode: str = "none") -> None:
@@ -788,18 +796,19 @@ def rms_norm(x: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tenso
     laid out like ``x``): ``gate_mode="silu_before"`` multiplies ``x`` by ``silu(gate)`` before
     the norm, ``"sigmoid_after"`` multiplies the result by ``sigmoid(gate)``, ``"silu_after"``
     by ``silu(gate)``. A ``weight`` shorter than a row repeats along it (its length must divide
-    a group's width: one weight shared by every head).
+    a group's width: one weight shared by every head); ``None``: no weight.
     """
     op = "rms_norm"
     if _left_out and op in _left_out:
         return
     _need(op, "x", x, torch.float32, 2)
-    _need(op, "weight", weight, torch.float32, 1)
+    if weight is not None:
+        _need(op, "weight", weight, torch.float32, 1)
     _need(op, "out", out, ndim=2)
     if out.dtype not in _TYPE:
         raise BackendError(f"{op}: out must be float32 or bfloat16, got {out.dtype}")
     width = out.shape[1]
-    period = 0 if weight.shape[0] == width else weight.shape[0]
+    period = 0 if weight is None or weight.shape[0] == width else weight.shape[0]
     if x.shape[1] != width or groups < 1 or width % groups or \
             (period and (width // groups) % period):
         raise BackendError(f"{op}: widths differ or {groups} groups do not divide {width}")
@@ -824,8 +833,9 @@ def rms_norm(x: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tenso
 
 
 def rope_frequencies(dims: int, base: float, device: torch.device,
-                     scaling: tuple[float, float, float, float] | None = None) -> torch.Tensor:
-    """``f_i = base^(-2i / dims)`` for the ``dims / 2`` pairs, as float64 on ``device`` (the
+                     scaling: tuple[float, float, float, float] | None = None,
+                     slowed: float = 1.0) -> torch.Tensor:
+    """``f_i = base^(-2i / dims) / slowed`` for the ``dims / 2`` pairs, as float64 on ``device`` (the
     kernels form ``position * f_i`` and its sine and cosine in double precision).
 
     ``scaling = (factor, low, high, original)`` rescales by wavelength ``l = 2 pi / f``: a
@@ -834,7 +844,7 @@ def rope_frequencies(dims: int, base: float, device: torch.device,
     the weight ``(original / l - low) / (high - low)`` on the kept one."""
     values = []
     for i in range(dims // 2):
-        f = float(base) ** (-2.0 * i / dims)
+        f = float(base) ** (-2.0 * i / dims) / slowed
         if scaling is not None:
             factor, low, high, original = scaling
             wavelength = 2.0 * math.pi / f
@@ -1481,9 +1491,13 @@ def moe_experts(hidden: torch.Tensor, w_in: torch.Tensor, w_out: torch.Tensor,
 
 
 def moe_join(pair_out: torch.Tensor, share: torch.Tensor, dst: torch.Tensor, *, top: int,
-             scale: torch.Tensor | None = None, accumulate: bool = True, rows: int) -> None:
+             scale: torch.Tensor | None = None, accumulate: bool = True, rows: int,
+             chosen: torch.Tensor | None = None, hidden: torch.Tensor | None = None,
+             experts: int = 0) -> None:
     """``dst[row] (+)= scale * sum_j share[row * top + j] * pair_out[row * top + j]`` in
-    float32, the choices in order; ``scale`` (float32 ``[width]``) is optional."""
+    float32, the choices in order; ``scale`` (float32 ``[width]``) is optional. With
+    ``hidden`` (the experts' input) and ``chosen``, a choice of ``experts`` or more is an
+    identity expert: ``hidden[row]`` stands for its ``pair_out``."""
     op = "moe_join"
     if _left_out and op in _left_out:
         return
@@ -1498,8 +1512,17 @@ def moe_join(pair_out: torch.Tensor, share: torch.Tensor, dst: torch.Tensor, *, 
         _need(op, "scale", scale, torch.float32, 1)
         if scale.shape[0] != width:
             raise BackendError(f"{op}: the scale does not match the width")
+    if hidden is not None:
+        _need(op, "hidden", hidden, ndim=2)
+        _need(op, "chosen", chosen, torch.int32, 1)
+        if hidden.dtype not in _TYPE or hidden.shape[1] != width or hidden.shape[0] < rows or \
+                chosen.shape[0] < rows * top or experts < 1:
+            raise BackendError(f"{op}: the identity experts' input does not match")
     status = library("moe").ayk_moe_join(
-        _ptr(pair_out), c_int(pair_out.stride(0)), _ptr(share), c_int(rows), c_int(top),
+        _ptr(pair_out), c_int(pair_out.stride(0)), _ptr(share),
+        _ptr(chosen if hidden is not None else None), _ptr(hidden),
+        c_int(0 if hidden is None else hidden.stride(0)), c_int(experts),
+        c_int(0 if hidden is None else _TYPE[hidden.dtype]), c_int(rows), c_int(top),
         _ptr(scale), _ptr(dst), c_int(dst.stride(0)), c_int(width),
         c_int(1 if accumulate else 0), _stream())
     check(status, op)
@@ -1507,13 +1530,16 @@ def moe_join(pair_out: torch.Tensor, share: torch.Tensor, dst: torch.Tensor, *, 
 
 def moe_route_scored(logits: torch.Tensor, chosen: torch.Tensor, share: torch.Tensor, *,
                      top: int, groups: int = 1, keep: int = 1, factor: float = 1.0,
-                     renormalise: bool = False, rows: int) -> None:
-    """Routing by scores ``s = sigmoid(logits)`` (float32 ``[N, experts]``): the experts form
-    ``groups`` equal groups of neighbours, a group's score is the sum of its two largest ``s``,
-    only experts of the ``keep`` best groups can be chosen, and of those the ``top`` largest
-    are (ties to the smaller index), in descending order, into ``chosen`` (int32 ``[N * top]``).
-    ``share`` (float32 ``[N * top]``) gets ``factor * s``, divided by the chosen ones' sum
-    with ``renormalise``."""
+                     renormalise: bool = False, rows: int, softmax: bool = False,
+                     correction: torch.Tensor | None = None, floor: float = 0.0) -> None:
+    """Routing by scores ``s = sigmoid(logits)`` (float32 ``[N, experts]``), or the softmax over
+    all experts with ``softmax``; what is compared is ``s + correction`` (float32
+    ``[experts]``, optional). The experts form ``groups`` equal groups of neighbours, a group's
+    score is the sum of its two largest, only experts of the ``keep`` best groups can be
+    chosen, and of those the ``top`` largest are (ties to the smaller index), in descending
+    order, into ``chosen`` (int32 ``[N * top]``). ``share`` (float32 ``[N * top]``) gets
+    ``factor * s`` without the correction, divided by the chosen ones' sum plus ``floor`` with
+    ``renormalise``."""
     op = "moe_route_scored"
     if _left_out and op in _left_out:
         return
@@ -1522,10 +1548,14 @@ def moe_route_scored(logits: torch.Tensor, chosen: torch.Tensor, share: torch.Te
     _need(op, "share", share, torch.float32, 1)
     if rows > logits.shape[0] or min(chosen.shape[0], share.shape[0]) < rows * top:
         raise BackendError(f"{op}: shapes do not fit")
+    if correction is not None:
+        _need(op, "correction", correction, torch.float32, 1)
+        if correction.shape[0] != logits.shape[1]:
+            raise BackendError(f"{op}: one correction per expert")
     status = library("moe").ayk_moe_route_scored(
         _ptr(logits), c_int(logits.stride(0)), c_int(rows), c_int(logits.shape[1]), c_int(top),
         c_int(groups), c_int(keep), c_float(factor), c_int(1 if renormalise else 0),
-        _ptr(chosen), _ptr(share), _stream())
+        c_int(1 if softmax else 0), _ptr(correction), c_float(floor), _ptr(chosen), _ptr(share), _stream())
     check(status, op)
 
 
@@ -1871,11 +1901,14 @@ def gated_attention_prepare(proj: torch.Tensor, *, k_offset: int, v_offset: int,
                             eps: float, slot_mapping: torch.Tensor | None,
                             k_pages: torch.Tensor | None, v_pages: torch.Tensor | None,
                             q: torch.Tensor, heads: int, kv_heads: int, dim: int, vdim: int,
-                            rows: int) -> None:
+                            rows: int, positions: torch.Tensor | None = None,
+                            freq: torch.Tensor | None = None, layout: str = "neighbours"
+                            ) -> None:
     """From a row of a fused projection (float32: ``heads * dim`` queries at 0, ``kv_heads *
     dim`` keys at ``k_offset``, ``kv_heads * vdim`` values at ``v_offset``): queries and keys
     each normalised by the root mean square over their whole projection with a weight per
-    entry (``None``: no norm), the queries written to ``q`` ``[N, heads * dim]``, the key and
+    entry (``None``: no norm), the first ``2 * len(freq)`` entries of every head rotated by the
+    row's position (``freq`` ``None``: no rotation; see :func:`rope`), the queries written to ``q`` ``[N, heads * dim]``, the key and
     value into the row's cache slot (``k_pages`` ``[page, kv_head, slot, dim]``, ``v_pages``
     likewise with ``vdim``; ``None``: stored nowhere)."""
     op = "gated_attention_prepare"
@@ -1907,12 +1940,19 @@ def gated_attention_prepare(proj: torch.Tensor, *, k_offset: int, v_offset: int,
     if rows > proj.shape[0] or rows > q.shape[0] or q.shape[1] != heads * dim or \
             proj.shape[1] < v_offset + kv_heads * vdim:
         raise BackendError(f"{op}: shapes do not fit")
+    rot_dims = 0 if freq is None else 2 * freq.shape[0]
+    if rot_dims:
+        _need(op, "freq", freq, torch.float64, 1)
+        _need(op, "positions", positions, torch.int32, 1)
+        if layout not in ROPE_LAYOUTS or rot_dims > dim or rows > positions.shape[0]:
+            raise BackendError(f"{op}: the rotation does not fit")
     status = library("gated_attention").ayk_gated_prepare(
         _ptr(proj), c_int(proj.stride(0)), c_int(k_offset), c_int(v_offset), _ptr(q_weight),
         _ptr(k_weight), c_float(eps), _ptr(slot_mapping if k_pages is not None else None),
         _ptr(k_pages), _ptr(v_pages), c_int(page_size), _ptr(q), c_int(q.stride(0)),
         c_int(rows), c_int(heads), c_int(kv_heads), c_int(dim), c_int(vdim),
-        c_int(_TYPE[q.dtype]), _stream())
+        _ptr(positions if rot_dims else None), _ptr(freq if rot_dims else None),
+        c_int(rot_dims), c_int(ROPE_LAYOUTS[layout]), c_int(_TYPE[q.dtype]), _stream())
     check(status, op)
 
 
@@ -2024,3 +2064,264 @@ def gated_decode(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor,
         _launches += 1  # the merge of the shares is a launch of its own
     check(status, op)
     return True
+
+
+# ---- linear attention with a matrix state per head ------------------------------------------
+
+DECAYS = {"fixed": 0, "head": 1, "channel": 2}
+HEAD_GATES = {"none": 0, "sigmoid": 1, "silu": 2}
+#: rows of a chunk (``LA_C`` in ``csrc/linear_attention.cu``)
+LINEAR_CHUNK = 16
+
+
+class _LinearArgs(Structure):
+    """``LinearArgs`` of ``csrc/linear_attention.cu``, field by field."""
+
+    _fields_ = [(name, c_void_p) for name in (
+        "in_", "raw", "decay_raw", "a_log", "dt_bias", "fixed", "freq", "positions", "row_start",
+        "state_slot", "state", "scratch", "out", "conv_weight", "decay_up", "gate_up",
+        "norm_weight", "gated")] + [("state_stride", c_longlong)] + [(name, c_int) for name in (
+            "ld_in", "ld_raw", "ld_decay", "ld_out", "ld_gated", "q_at", "k_at", "v_at",
+            "decay_at", "beta_at", "gate_at", "heads", "kv_heads", "N", "P", "taps", "channels",
+            "ring_at", "decay_mode", "delta", "unit", "gate_mode", "decay_rank", "gate_rank",
+            "rot_dims", "rot_layout", "requests", "chunks")] + [(name, c_float) for name in (
+                "q_scale", "k_scale", "eps", "unit_eps")]
+
+
+@dataclass(frozen=True, slots=True)
+class LinearShape:
+    """What a layer of linear attention is (see ``csrc/linear_attention.cu``): per head a state
+    ``S`` of ``dim`` key channels by ``columns``; ``decay`` ``"fixed"`` (one number per head),
+    ``"head"`` or ``"channel"`` (``exp(-exp(a_log) * softplus(raw + dt_bias))``); ``delta``: what
+    is written is ``beta (v - S^T k)`` with ``beta = sigmoid(raw)``, else ``v``; ``unit``: queries
+    and keys divided by ``sqrt(x . x + unit_eps)``; then ``q_scale`` and ``k_scale``; ``taps`` > 0:
+    a causal convolution with silu on queries, keys and values first; ``gate``: the factor on
+    the normed heads (``none``, ``sigmoid``, ``silu``); ``decay_rank`` / ``gate_rank`` > 0: a second,
+    stored matrix turns that many columns of the projection into the raw decays or gates.
+
+    ``q_at`` .. ``gate_at`` are columns of the fused projection."""
+
+    heads: int
+    kv_heads: int
+    dim: int
+    columns: int
+    decay: str
+    delta: bool
+    unit: bool
+    gate: str
+    q_at: int
+    k_at: int
+    v_at: int
+    gate_at: int
+    decay_at: int = 0
+    beta_at: int = 0
+    taps: int = 0
+    decay_rank: int = 0
+    gate_rank: int = 0
+    q_scale: float = 1.0
+    k_scale: float = 1.0
+    eps: float = 1e-6
+    unit_eps: float = 1e-6
+    rot_layout: str = "halves"
+
+    @property
+    def channels(self) -> int:
+        """Channels of the convolution: queries, keys and values side by side."""
+        return 2 * self.kv_heads * self.dim + self.heads * self.columns
+
+    @property
+    def ring_at(self) -> int:
+        """Floats of a request's state ahead of its convolution's ring."""
+        return self.heads * self.dim * self.columns
+
+    @property
+    def state_floats(self) -> int:
+        """Floats of a request's state, a multiple of four."""
+        return -(-(self.ring_at + self.taps * self.channels) // 4) * 4
+
+
+def conv_ring(x: torch.Tensor, weight: torch.Tensor, state: torch.Tensor, out: torch.Tensor, *,
+              ring_at: int, request_of_row: torch.Tensor, row_start: torch.Tensor,
+              state_slot: torch.Tensor, positions: torch.Tensor, rows: int) -> None:
+    """``out = silu(causal convolution of x per channel)`` for the step's rows (float32 ``[N,
+    channels]``; ``weight`` ``[channels, taps]``, its last column the current row's). The inputs
+    ahead of a request's first row come from the ring ``state[slot, ring_at:]`` (``[taps,
+    channels]``, position ``p`` at ``p % taps``), which takes up the step's last inputs: one
+    launch."""
+    op = "conv_ring"
+    if _left_out and op in _left_out:
+        return
+    _need(op, "x", x, torch.float32, 2)
+    _need(op, "weight", weight, torch.float32, 2)
+    _need(op, "state", state, torch.float32, 2)
+    _need(op, "out", out, torch.float32, 2)
+    for name, tensor in (("request_of_row", request_of_row), ("row_start", row_start),
+                         ("state_slot", state_slot), ("positions", positions)):
+        _need(op, name, tensor, torch.int32, 1)
+    channels, taps = weight.shape
+    if x.shape[1] != channels or out.shape[1] != channels or rows > x.shape[0] or \
+            rows > out.shape[0] or state.shape[1] < ring_at + taps * channels or \
+            not weight.is_contiguous() or rows > positions.shape[0] or \
+            rows > request_of_row.shape[0]:
+        raise BackendError(f"{op}: shapes do not fit")
+    status = library("linear_attention").ayk_conv_ring(
+        _ptr(x), c_int(x.stride(0)), _ptr(weight), c_void_p(state.data_ptr() + 4 * ring_at),
+        c_longlong(state.stride(0)), _ptr(request_of_row), _ptr(row_start), _ptr(state_slot),
+        _ptr(positions), _ptr(out), c_int(out.stride(0)), c_int(rows), c_int(channels),
+        c_int(taps), _stream())
+    check(status, op)
+
+
+def _linear_args(op: str, shape: LinearShape, state: torch.Tensor, state_slot: torch.Tensor,
+                 positions: torch.Tensor, a_log: torch.Tensor | None,
+                 dt_bias: torch.Tensor | None, fixed: torch.Tensor | None,
+                 freq: torch.Tensor | None) -> _LinearArgs:
+    _need(op, "state", state, torch.float32, 2)
+    _need(op, "state_slot", state_slot, torch.int32, 1)
+    _need(op, "positions", positions, torch.int32, 1)
+    for name, tensor, size in (
+            ("fixed", fixed, shape.heads if shape.decay == "fixed" else None),
+            ("a_log", a_log, shape.heads if shape.decay != "fixed" else None),
+            ("dt_bias", dt_bias, {"head": shape.heads, "channel": shape.heads * shape.dim}.get(
+                shape.decay))):
+        if size is not None:
+            if tensor is None:
+                raise BackendError(f"{op}: {name} is missing")
+            _need(op, name, tensor, torch.float32, 1)
+            if tensor.shape[0] != size:
+                raise BackendError(f"{op}: {name} must hold {size} entries")
+    if state.shape[1] < shape.ring_at + shape.taps * shape.channels:
+        raise BackendError(f"{op}: the state is too small")
+    rot_dims = 0 if freq is None else 2 * freq.shape[0]
+    if rot_dims:
+        _need(op, "freq", freq, torch.float64, 1)
+    if sizeof(_LinearArgs) != library("linear_attention").ayk_linear_args_bytes():
+        raise BackendError(f"{op}: the argument struct does not match the library's")
+    args = _LinearArgs()
+    args.a_log, args.dt_bias, args.fixed = _address(a_log), _address(dt_bias), _address(fixed)
+    args.freq = _address(freq if rot_dims else None)
+    args.positions, args.state_slot = _address(positions), _address(state_slot)
+    args.state, args.state_stride = _address(state), state.stride(0)
+    args.q_at, args.k_at, args.v_at = shape.q_at, shape.k_at, shape.v_at
+    args.decay_at, args.beta_at, args.gate_at = shape.decay_at, shape.beta_at, shape.gate_at
+    args.heads, args.kv_heads, args.N, args.P = (shape.heads, shape.kv_heads, shape.dim,
+                                                 shape.columns)
+    args.taps, args.channels, args.ring_at = shape.taps, shape.channels, shape.ring_at
+    args.decay_mode, args.delta, args.unit = DECAYS[shape.decay], int(shape.delta), int(shape.unit)
+    args.gate_mode = HEAD_GATES[shape.gate]
+    args.decay_rank, args.gate_rank = shape.decay_rank, shape.gate_rank
+    args.rot_dims, args.rot_layout = rot_dims, ROPE_LAYOUTS[shape.rot_layout]
+    args.q_scale, args.k_scale = shape.q_scale, shape.k_scale
+    args.eps, args.unit_eps = shape.eps, shape.unit_eps
+    return args
+
+
+def _address(tensor: torch.Tensor | None) -> int | None:
+    return None if tensor is None else tensor.data_ptr()
+
+
+def linear_chunks(host_rows: list[int]) -> int:
+    """Chunks :func:`linear_attention_chunks` cuts a step of these row counts into."""
+    return sum(-(-rows // LINEAR_CHUNK) for rows in host_rows)
+
+
+def linear_chunk_floats(shape: LinearShape) -> int:
+    """Scratch floats per chunk (all heads) of :func:`linear_attention_chunks`."""
+    pad = -(-shape.dim // 4) * 4
+    return shape.heads * (3 * LINEAR_CHUNK * shape.dim + pad + LINEAR_CHUNK * LINEAR_CHUNK)
+
+
+def linear_attention_chunks(qkv: torch.Tensor, proj: torch.Tensor, shape: LinearShape,
+                            state: torch.Tensor, out: torch.Tensor, scratch: torch.Tensor, *,
+                            q_at: int, k_at: int, v_at: int, row_start: torch.Tensor,
+                            state_slot: torch.Tensor, positions: torch.Tensor,
+                            host_rows: list[int], decay_raw: torch.Tensor | None = None,
+                            a_log: torch.Tensor | None = None,
+                            dt_bias: torch.Tensor | None = None,
+                            fixed: torch.Tensor | None = None,
+                            freq: torch.Tensor | None = None) -> None:
+    """The recurrence of ``shape`` over the step's rows, request by request, from and into each
+    request's slot of ``state``, in chunks of ``LINEAR_CHUNK`` rows (two launches): ``out``
+    (float32 ``[N, heads * columns]``) gets ``S^T q`` per head, before any norm. ``qkv``
+    (float32) holds queries, keys and values at columns ``q_at``, ``k_at``, ``v_at`` (after the
+    convolution where there is one); ``proj`` the projection's rows, whose ``decay_at`` (decay
+    ``"head"``) and ``beta_at`` columns are read; ``decay_raw`` (float32 ``[N, heads * dim]``)
+    the raw decays of decay ``"channel"``. ``scratch``: float32, contiguous, at least
+    ``linear_chunks(host_rows) * linear_chunk_floats(shape)`` elements."""
+    op = "linear_attention_chunks"
+    if _left_out and op in _left_out:
+        return
+    _need(op, "qkv", qkv, torch.float32, 2)
+    _need(op, "proj", proj, torch.float32, 2)
+    _need(op, "out", out, torch.float32, 2)
+    _need(op, "scratch", scratch, torch.float32)
+    _need(op, "row_start", row_start, torch.int32, 1)
+    args = _linear_args(op, shape, state, state_slot, positions, a_log, dt_bias, fixed, freq)
+    rows, requests, chunks = sum(host_rows), len(host_rows), linear_chunks(host_rows)
+    if rows > min(qkv.shape[0], proj.shape[0], out.shape[0], positions.shape[0]) or \
+            row_start.shape[0] < requests + 1 or state_slot.shape[0] < requests or \
+            not scratch.is_contiguous() or \
+            scratch.numel() < chunks * linear_chunk_floats(shape):
+        raise BackendError(f"{op}: shapes do not fit")
+    if shape.decay == "channel":
+        _need(op, "decay_raw", decay_raw, torch.float32, 2)
+        if decay_raw.shape[0] < rows or decay_raw.shape[1] < shape.heads * shape.dim:
+            raise BackendError(f"{op}: the raw decays do not match")
+        args.decay_raw, args.ld_decay = decay_raw.data_ptr(), decay_raw.stride(0)
+    args.in_, args.ld_in = qkv.data_ptr(), qkv.stride(0)
+    args.raw, args.ld_raw = proj.data_ptr(), proj.stride(0)
+    args.q_at, args.k_at, args.v_at = q_at, k_at, v_at
+    args.row_start, args.requests, args.chunks = row_start.data_ptr(), requests, chunks
+    args.scratch, args.out, args.ld_out = scratch.data_ptr(), out.data_ptr(), out.stride(0)
+    global _launches
+    _launches += 1  # the chunks' matrices, then the scan
+    check(library("linear_attention").ayk_linear_chunks(byref(args), _stream()), op)
+
+
+def linear_attention_decode(proj: torch.Tensor, shape: LinearShape, state: torch.Tensor,
+                            out: torch.Tensor, *, state_slot: torch.Tensor,
+                            positions: torch.Tensor, rows: int,
+                            conv_weight: torch.Tensor | None = None,
+                            a_log: torch.Tensor | None = None,
+                            dt_bias: torch.Tensor | None = None,
+                            decay_up: torch.Tensor | None = None,
+                            gate_up: torch.Tensor | None = None,
+                            norm_weight: torch.Tensor | None = None,
+                            fixed: torch.Tensor | None = None,
+                            freq: torch.Tensor | None = None) -> None:
+    """A step of single rows (row ``r`` is request ``r``'s) in one launch, from the projection's
+    rows (float32) to ``out`` (compute type, ``[N, heads * columns]``): convolution, low-rank
+    decays and gates, rotation, unit keys, the state's update, ``S^T q``, each head divided by
+    its root mean square, times ``norm_weight`` (float32 ``[columns]``, optional) and the gate."""
+    op = "linear_attention_decode"
+    if _left_out and op in _left_out:
+        return
+    _need(op, "proj", proj, torch.float32, 2)
+    _need(op, "out", out, ndim=2)
+    args = _linear_args(op, shape, state, state_slot, positions, a_log, dt_bias, fixed, freq)
+    if out.dtype not in _TYPE or rows > min(proj.shape[0], out.shape[0], positions.shape[0],
+                                            state_slot.shape[0]) or \
+            out.shape[1] != shape.heads * shape.columns:
+        raise BackendError(f"{op}: shapes do not fit")
+    for name, tensor, size in (
+            ("conv_weight", conv_weight, (shape.channels, shape.taps) if shape.taps else None),
+            ("decay_up", decay_up, (shape.heads * shape.dim, shape.decay_rank)
+             if shape.decay_rank else None),
+            ("gate_up", gate_up, (shape.heads * shape.columns, shape.gate_rank)
+             if shape.gate_rank else None)):
+        if size is not None:
+            _need(op, name, tensor, torch.float32 if name == "conv_weight" else out.dtype, 2)
+            if tuple(tensor.shape) != size or not tensor.is_contiguous():  # type: ignore
+                raise BackendError(f"{op}: {name} must be contiguous {list(size)}")
+    if norm_weight is not None:
+        _need(op, "norm_weight", norm_weight, torch.float32, 1)
+        if norm_weight.shape[0] != shape.columns:
+            raise BackendError(f"{op}: norm_weight must hold {shape.columns} entries")
+    args.in_, args.ld_in = proj.data_ptr(), proj.stride(0)
+    args.conv_weight = _address(conv_weight if shape.taps else None)
+    args.decay_up = _address(decay_up if shape.decay_rank else None)
+    args.gate_up = _address(gate_up if shape.gate_rank else None)
+    args.norm_weight, args.gated, args.ld_gated = (_address(norm_weight), out.data_ptr(),
+                                                   out.stride(0))
+    check(library("linear_attention").ayk_linear_decode(
+        byref(args), c_int(rows), c_int(_TYPE[out.dtype]), _stream()), op)

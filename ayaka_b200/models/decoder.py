@@ -21,7 +21,12 @@ class DecoderModel(Part):
     """Embedding -> runs of blocks -> final norm on the wanted rows -> head (fp32 logits).
 
     Parameter names: ``embedding.weight``, ``position.*``, ``layers.<i>.<part>.*``,
-    ``final_norm.*`` and, when the head is not tied, ``head.weight``.
+    ``final_norm.*``, when the head is not tied ``head.weight`` and, with an entry part,
+    ``entry.*``.
+
+    A layer that the order names more than once runs with the same weights each time and has a
+    cache or state per run. With ``spec.entry`` the runs that open a pass
+    (``Run.opens_pass``) are preceded by that part, which is shown the embeddings once a step.
     """
 
     def __init__(self, spec: ModelSpec, ctx: BuildContext) -> None:
@@ -42,6 +47,11 @@ class DecoderModel(Part):
             "final_norm", build_part("norm", spec.final_norm.kind, spec.final_norm, ctx))
         self.head = self.add_child(
             "head", build_part("head", spec.head.kind, spec.head, ctx, self.embedding))
+        self.entry = None if spec.entry is None else self.add_child(
+            "entry", build_part("entry", spec.entry.kind, spec.entry, ctx))
+        self._opens = any(run.opens_pass is not None for run in spec.order)
+        if self._opens and self.entry is None:
+            raise ValueError("an order that opens passes needs an entry part")
         for position, run in enumerate(spec.order):
             if not 0 <= run.layer < len(self.blocks):
                 raise ValueError(f"order[{position}] names layer {run.layer}, which does not "
@@ -87,7 +97,9 @@ class DecoderModel(Part):
         self.embedding.forward(  # type: ignore[attr-defined]
             step, residual, self.position.added_rows(step))  # type: ignore[attr-defined]
         step.extra.pop("block.stream_copy", None)  # (a block's copy of an earlier stream)
-        runs = self._native_runs(step, caches) if ops.NATIVE_STEP else None
+        if self._opens:
+            self.entry.begin(residual, step)  # type: ignore[union-attr]
+        runs = self._native_runs(step, caches) if ops.NATIVE_STEP and not self._opens else None
         if runs is not None:
             # every layer can run from the C++ host code: one call walks the whole order
             native.run_layers(runs, native.step_args(step, residual.device), residual)
@@ -96,7 +108,12 @@ class DecoderModel(Part):
             for index, run in enumerate(spec.order):
                 # a block that can apply the next layer's first norm on its way out is told
                 # which one that is (and says so in ``step.extra["block.normed_by"]``)
-                following = spec.order[index + 1].layer if index + 1 < len(spec.order) else None
+                # (ahead of a pass the stream changes once more: no norm can be applied early)
+                if run.opens_pass is not None:
+                    self.entry.forward(residual, step, run.opens_pass)  # type: ignore
+                after = spec.order[index + 1] if index + 1 < len(spec.order) else None
+                following = after.layer if after is not None and after.opens_pass is None \
+                    else None
                 step.extra["block.next_norm"] = None if following is None else getattr(
                     self.blocks[following], "mixer_norm", None)
                 self.blocks[run.layer].forward(residual, step, caches[index])  # type: ignore

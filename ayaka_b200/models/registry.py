@@ -83,3 +83,4 @@ def _builtin() -> None:
     import ayaka_b200.models.mapuvik  # noqa: F401
     import ayaka_b200.models.rizitar  # noqa: F401
     import ayaka_b200.models.semadra  # noqa: F401
+    import ayaka_b200.models.senurax  # noqa: F401

@@ -112,14 +112,14 @@ class Part:
 
 _REGISTRIES: dict[str, dict[str, Callable[..., Part]]] = {
     "mixer": {}, "feed_forward": {}, "norm": {}, "position": {}, "block": {}, "embedding": {},
-    "head": {}, "side": {},
+    "head": {}, "side": {}, "entry": {},
 }
 
 
 def register_part(family: str, kind: str) -> Callable[[Callable[..., Part]], Callable[..., Part]]:
     """Class decorator: make ``kind`` buildable in ``family`` (``mixer``, ``feed_forward``,
-    ``norm``, ``position``, ``block``, ``embedding``, ``head``, ``side``). Registering a kind again
-    replaces it, so a test may define a toy part without touching the package."""
+    ``norm``, ``position``, ``block``, ``embedding``, ``head``, ``side``, ``entry``). Registering a
+    kind again replaces it, so a test may define a toy part without touching the package."""
     if family not in _REGISTRIES:
         raise ConfigError("parts.family", "INVALID_CHOICE",
                           f"unknown family {family!r}; families are {sorted(_REGISTRIES)}")

@@ -13,6 +13,9 @@ from ayaka_b200.parts.spec import PartSpec
 
 __all__ = ["MixtureOfExperts"]
 
+#: added to the chosen experts' sum before it divides (``softmax_corrected``)
+WEIGHT_FLOOR = 1e-20
+
 
 @register_part("feed_forward", "experts")
 class MixtureOfExperts(FeedForward):
@@ -41,10 +44,17 @@ class MixtureOfExperts(FeedForward):
     ``unit="relu_squared"`` an expert has no gate: ``W_down relu(W_up h)^2``, and ``in.weight``
     is ``[experts * inner, width]``.
 
+    With ``scoring="softmax_corrected"`` the scores are the softmax over all experts, the ``top``
+    largest ``s + correction`` (a learned vector) are chosen, and the weights are
+    ``route_scale * s / (sum of the chosen s + 1e-20)``. With ``identity`` the router has that
+    many outputs more, which stand for identity experts: one that is chosen contributes the
+    row's input ``h`` itself, times its weight, and has no matrices.
+
     Spec parameters: ``width``, ``experts``, ``top``, ``inner``; ``unit`` (``clamped`` when
     absent, with ``limit`` and ``alpha``; or ``silu``; or ``relu_squared``); ``scoring``
-    (``softmax`` when absent; ``softmax_all``; or ``sigmoid`` with ``groups``, ``keep_groups``,
-    ``route_scale``, ``renormalise``); ``shared_inner`` (0 when absent).
+    (``softmax`` when absent; ``softmax_all``; ``softmax_corrected`` with ``route_scale``; or
+    ``sigmoid`` with ``groups``, ``keep_groups``, ``route_scale``, ``renormalise``); ``identity`` and
+    ``shared_inner`` (0 when absent).
     """
 
     def __init__(self, spec: PartSpec, ctx: BuildContext) -> None:
@@ -63,23 +73,30 @@ class MixtureOfExperts(FeedForward):
             self.shift = 1.0
         else:
             raise ValueError(f"unknown expert unit {self.unit!r}")
-        if not 1 <= self.top <= self.experts <= 1024 or self.inner < 1 or not self.limit > 0:
-            raise ValueError("experts takes 1 <= top <= experts <= 1024, inner >= 1 and a "
-                             "positive limit")
+        self.identity = int(spec.get("identity", 0))  # type: ignore[arg-type]
+        self.outputs = self.experts + self.identity  # of the router
+        if not 1 <= self.top <= self.outputs or not 1 <= self.experts or self.identity < 0 or \
+                self.outputs > 1024 or self.inner < 1 or not self.limit > 0:
+            raise ValueError("experts takes 1 <= top <= experts + identity <= 1024, inner >= 1 "
+                             "and a positive limit")
         self.scoring = str(spec.get("scoring", "softmax"))
         self.groups = int(spec.get("groups", 1))  # type: ignore[arg-type]
         self.keep_groups = int(spec.get("keep_groups", self.groups))  # type: ignore[arg-type]
         self.route_scale = float(spec.get("route_scale", 1.0))  # type: ignore[arg-type]
         self.renormalise = bool(spec.get("renormalise", False))
-        if self.scoring not in ("softmax", "softmax_all", "sigmoid"):
+        if self.scoring not in ("softmax", "softmax_all", "softmax_corrected", "sigmoid"):
             raise ValueError(f"unknown router scoring {self.scoring!r}")
+        if self.identity and self.scoring == "sigmoid":
+            raise ValueError("identity experts come with a softmax router")
         if self.scoring == "sigmoid" and (
                 self.groups < 1 or self.experts % self.groups
                 or not 1 <= self.keep_groups <= self.groups
                 or self.top > self.keep_groups * (self.experts // self.groups)):
             raise ValueError("groups must divide experts, 1 <= keep_groups <= groups, and the "
                              "kept groups must hold at least top experts")
-        self.router = self.add_param("router.weight", (self.experts, self.width), "matrix")
+        self.router = self.add_param("router.weight", (self.outputs, self.width), "matrix")
+        self.correction = self.add_param("correction", (self.outputs,), "vector") \
+            if self.scoring == "softmax_corrected" else None
         self.in_weight = self.add_param(
             "in.weight", (self.experts * (1 if self.single else 2) * self.inner, self.width),
             "matrix")
@@ -108,7 +125,7 @@ class MixtureOfExperts(FeedForward):
         # scratch for the largest step, so that its addresses never change
         most = work.max_rows
         places, tiles = ops.moe_scratch(most, self.experts, top)
-        logits = work.buffer("experts.logits", self.experts, torch.float32)
+        logits = work.buffer("experts.logits", self.outputs, torch.float32)
         chosen = work.buffer("experts.chosen", top, torch.int32).view(-1)
         share = work.buffer("experts.share", top, torch.float32).view(-1)
         sorted_pairs = work.buffer("experts.sorted", 1, torch.int32, rows=places).view(-1)
@@ -120,6 +137,10 @@ class MixtureOfExperts(FeedForward):
             ops.moe_route_scored(logits, chosen, share, top=top, groups=self.groups,
                                  keep=self.keep_groups, factor=self.route_scale,
                                  renormalise=self.renormalise, rows=n)
+        elif self.correction is not None:
+            ops.moe_route_scored(logits, chosen, share, top=top, factor=self.route_scale,
+                                 renormalise=True, rows=n, softmax=True,
+                                 correction=self.correction, floor=WEIGHT_FLOOR)
         else:
             ops.moe_route(logits, chosen, share, top=top, rows=n,
                           over_all=self.scoring == "softmax_all")
@@ -127,7 +148,9 @@ class MixtureOfExperts(FeedForward):
                         experts=self.experts, top=top, limit=self.limit, alpha=self.alpha,
                         shift=self.shift, sorted_pairs=sorted_pairs, tile_expert=tile_expert,
                         inner=inner, rows=n, single=self.single)
+        identity = dict(chosen=chosen, hidden=hidden, experts=self.experts) \
+            if self.identity else {}
         ops.moe_join(pair_out, share, residual, top=top, scale=scale, accumulate=accumulate,
-                     rows=n)
+                     rows=n, **identity)
         if self.shared is not None:
             self.shared.forward(hidden, residual, step)  # type: ignore[attr-defined]

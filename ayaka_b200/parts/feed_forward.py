@@ -42,8 +42,8 @@ class DenseMLP(FeedForward):
     (parameter ``act.numbers`` = ``(p, q)``): the first product writes fp32, one element-wise
     launch adds the bias and applies the unit.
 
-    Spec parameters: ``width``, ``inner``, ``activation`` (``gelu_tanh``, ``gelu_erf`` or
-    ``xielu``), ``bias`` (bool).
+    Spec parameters: ``width``, ``inner``, ``activation`` (``gelu_tanh``, ``gelu_erf``,
+    ``relu_squared`` or ``xielu``), ``bias`` (bool).
     """
 
     def __init__(self, spec: PartSpec, ctx: BuildContext) -> None:

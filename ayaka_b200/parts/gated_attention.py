@@ -1,4 +1,4 @@
-"""Softmax attention with a window that keeps the first tokens, and an output gate."""
+"""Softmax attention with rotated heads, a window that keeps the first tokens, an output gate."""
 
 from __future__ import annotations
 
@@ -15,20 +15,24 @@ __all__ = ["GatedAttention"]
 
 @register_part("mixer", "gated_attention")
 class GatedAttention(Mixer):
-    """Grouped softmax attention over paged keys and values, without positions in its scores.
+    """Grouped softmax attention over paged keys and values.
 
     One fused projection gives queries (``num_heads x head_dim``), keys (``num_kv_heads x
     head_dim``), values (``num_kv_heads x value_dim``) and, with ``gate``, one raw gate per
     entry of the joined heads. With ``qk_norm`` the whole query projection and the whole key
     projection are each normalised by their root mean square (all heads at once, a plain weight
-    per entry). Query head ``h`` uses key/value head ``h // (num_heads / num_kv_heads)``;
-    ``score = scale * q . k``; the query at position ``p`` sees key ``j <= p`` when
-    ``p - j < window`` (``window`` 0: every earlier key) or ``j < keep_first``: the sequence's
-    first tokens stay in sight at their true positions; softmax in fp32; the joined heads are
-    multiplied entry by entry by ``sigmoid(gate)``; then the output projection.
+    per entry). With ``rot_dims`` the first so many entries of every query and key head are
+    rotated by the position (``rot_layout``, frequencies ``rot_base^(-2i/rot_dims) / rot_slowed``);
+    without, the scores know no positions. Query head ``h`` uses key/value head
+    ``h // (num_heads / num_kv_heads)``; ``score = scale * q . k``; the query at position ``p`` sees
+    key ``j <= p`` when ``p - j < window`` (``window`` 0: every earlier key) or ``j < keep_first``:
+    the sequence's first tokens stay in sight at their true positions; softmax in fp32; with
+    ``gate`` the joined heads are multiplied entry by entry by its sigmoid; then the output
+    projection.
 
     Spec parameters: ``width``, ``num_heads``, ``num_kv_heads``, ``head_dim``, ``value_dim``,
-    ``scale``, ``window``, ``keep_first``, ``qk_norm``, ``eps``, ``gate``.
+    ``scale``, ``window``, ``keep_first``, ``qk_norm``, ``eps``, ``gate``, ``rot_dims``,
+    ``rot_base``, ``rot_slowed``, ``rot_layout``.
     """
 
     def __init__(self, spec: PartSpec, ctx: BuildContext, position: Part | None = None) -> None:
@@ -43,6 +47,13 @@ class GatedAttention(Mixer):
         self.keep_first = int(spec.get("keep_first", 0))  # type: ignore[arg-type]
         self.eps = float(spec.get("eps", 1e-6))  # type: ignore[arg-type]
         self.gated = bool(spec.get("gate", False))
+        self.rot_dims = int(spec.get("rot_dims", 0))  # type: ignore[arg-type]
+        self.rot_base = float(spec.get("rot_base", 10000.0))  # type: ignore[arg-type]
+        self.rot_slowed = float(spec.get("rot_slowed", 1.0))  # type: ignore[arg-type]
+        self.rot_layout = str(spec.get("rot_layout", "neighbours"))
+        self._freq: torch.Tensor | None = None
+        if self.rot_dims % 2 or not 0 <= self.rot_dims <= dim:
+            raise ValueError(f"rot_dims must be even and at most head_dim ({dim})")
         if heads < 1 or kv_heads < 1 or heads % kv_heads:
             raise ValueError(f"num_kv_heads ({kv_heads}) must divide num_heads ({heads})")
         if dim < 1 or vdim < 1 or self.window < 0 or self.keep_first < 0:
@@ -80,13 +91,17 @@ class GatedAttention(Mixer):
         proj = work.buffer("gated_attention.proj", self.proj_weight.shape[0], torch.float32)
         q = work.buffer("gated_attention.q", self.q_width, dtype)
         attended = work.buffer("gated_attention.out", self.out_width, dtype)
+        if self.rot_dims and self._freq is None:
+            self._freq = ops.rope_frequencies(self.rot_dims, self.rot_base, hidden.device,
+                                              slowed=self.rot_slowed)
         ops.linear(hidden, self.proj_weight, None, proj, rows=n)
         ops.gated_attention_prepare(
             proj, k_offset=self.q_width, v_offset=self.q_width + self.k_width,
             q_weight=self.q_norm, k_weight=self.k_norm, eps=self.eps,
             slot_mapping=group.slot_mapping, k_pages=cache.k_pages if cache.writes else None,
             v_pages=cache.v_pages if cache.writes else None, q=q, heads=self.num_heads,
-            kv_heads=self.num_kv_heads, dim=self.head_dim, vdim=self.value_dim, rows=n)
+            kv_heads=self.num_kv_heads, dim=self.head_dim, vdim=self.value_dim, rows=n,
+            positions=step.positions, freq=self._freq, layout=self.rot_layout)
         gate = proj[:, self.qkv_width:] if self.gated else None
         # Prompt portions in bfloat16, where the sizes are the tensor-core kernel's: the
         # engine's flash kernel, told of the kept keys, the value size and the gate. Single

@@ -81,10 +81,13 @@ class Run:
         layer: index into ``ModelSpec.layers``; a layer may appear in several runs.
         reads_cache_of: index of an earlier entry of the order whose cache this run reads
             instead of writing one of its own, or ``None``.
+        opens_pass: the number of the pass (0, 1, ...) over looped layers that starts with this
+            run: the model's ``entry`` part changes the stream ahead of it. ``None``: none does.
     """
 
     layer: int
     reads_cache_of: int | None = None
+    opens_pass: int | None = None
 
 
 @dataclass(frozen=True, slots=True)
@@ -101,4 +104,6 @@ class ModelSpec:
     final_norm: PartSpec
     head: PartSpec
     eos_token_id: int | None = None
+    #: the part of family ``entry`` that runs ahead of every pass (see ``Run.opens_pass``)
+    entry: PartSpec | None = None
     extra: Mapping[str, object] = field(default_factory=dict)
