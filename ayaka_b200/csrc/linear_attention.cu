@@ -78,8 +78,9 @@ __device__ __forceinline__ float la_silu(float z) { return z / (1.f + expf(-z));
 __device__ __forceinline__ float la_softplus(float z) {  // log(1 + e^z), for any z
   return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z)));
 }
-__device__ __forceinline__ float la_decay(float a_log, float raw) {
-  return expf(-expf(a_log) * la_softplus(raw));
+// a decay; rate = -exp(A_log)
+__device__ __forceinline__ float la_decay(float rate, float raw) {
+  return expf(rate * la_softplus(raw));
 }
 __device__ __forceinline__ void la_sincos(int position, double f, float& s, float& c) {
   // the angle and its reduction to [-pi, pi] in double precision (see rope.cuh)
@@ -108,6 +109,27 @@ la_conv_kernel(const float* __restrict__ in, int ld_in, const float* __restrict_
   for (int l = 0; l < TAPS; ++l) wv[l] = l < taps ? w[(size_t)c * taps + taps - 1 - l] : 0.f;
   pdl_wait_for(in, ring);
   const int first = blockIdx.x * LA_CONV_ROWS, last = min(rows, first + LA_CONV_ROWS);
+  if (TAPS <= 4 && last - first == LA_CONV_ROWS) {
+    // the usual case, all rows well inside one request: every input is fetched once
+    const int b = request_of_row[first];
+    if (b >= 0 && b == request_of_row[last - 1] && state_slot[b] >= 0 &&
+        first - row_start[b] >= taps - 1) {
+      float u[LA_CONV_ROWS + TAPS - 1];
+#pragma unroll
+      for (int i = 0; i < LA_CONV_ROWS + TAPS - 1; ++i) {
+        const int r = first + i - (TAPS - 1);
+        u[i] = r >= first - (taps - 1) ? in[(size_t)r * ld_in + c] : 0.f;
+      }
+#pragma unroll
+      for (int i = 0; i < LA_CONV_ROWS; ++i) {
+        float acc = 0.f;
+#pragma unroll
+        for (int l = 0; l < TAPS; ++l) acc = fmaf(wv[l], u[i + TAPS - 1 - l], acc);
+        out[(size_t)(first + i) * ld_out + c] = la_silu(acc);
+      }
+      return;
+    }
+  }
   for (int r = first; r < last; ++r) {
     const int b = request_of_row[r];
     if (b < 0 || state_slot[b] < 0) continue;
@@ -175,20 +197,22 @@ __device__ __forceinline__ bool la_find_chunk(const int* row_start, int requests
   return false;
 }
 
-// grid (chunks, heads). Shared memory: k, q, g and D_(C-1) k as [C][N].
-template <int NREG>  // ceil(N / 32)
+// grid (chunks, heads). Shared memory: k, q, g and D_(C-1) k as [C][NS], NS = N padded to a
+// multiple of 4 (the padding holds k = q = 0, g = 1). This kernel lets the scan start only when it
+// has ended: CTAs of the scan that took their places beside it would crowd on the SMs that empty
+// first, two or three on one (measured: 190 instead of 90 microseconds for 128 CTAs).
+template <int NREG, bool CHANNEL>  // ceil(N / 32); a decay per channel, or one per row
 __global__ void __launch_bounds__(LA_THREADS)
 la_prepare_kernel(const LinearArgs a) {
   extern __shared__ __align__(16) float la_smem[];
   __shared__ __align__(16) float A[LA_C][LA_C], B[LA_C][LA_C], T[LA_C][LA_C];
   __shared__ float beta_s[LA_C];
-  pdl_launch_dependents();
-  const int N = a.N, h = blockIdx.y, kv = h / (a.heads / a.kv_heads), tid = threadIdx.x;
-  const int lane = tid & 31, warp = tid >> 5;
+  const int N = a.N, NS = la_pad4(N), h = blockIdx.y, kv = h / (a.heads / a.kv_heads);
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   float* k_s = la_smem;
-  float* q_s = k_s + LA_C * N;
-  float* g_s = q_s + LA_C * N;
-  float* w_s = g_s + LA_C * N;
+  float* q_s = k_s + LA_C * NS;
+  float* g_s = q_s + LA_C * NS;
+  float* w_s = g_s + LA_C * NS;
   int b, t0, count;
   const bool found = la_find_chunk(a.row_start, a.requests, blockIdx.x, b, t0, count);
   const float* in = a.in;
@@ -198,64 +222,92 @@ la_prepare_kernel(const LinearArgs a) {
   pdl_wait_for(in, raw, decay_raw, scratch);
   if (!found) return;
   const int r0 = a.row_start[b] + t0;
-  const float a_log = a.decay_mode == DECAY_FIXED ? 0.f : a.a_log[h];
-  for (int idx = tid; idx < LA_C * N; idx += LA_THREADS) {
-    const int i = idx / N, n = idx - i * N;
-    float k = 0.f, q = 0.f, g = 1.f;
-    if (i < count) {
-      const float* row = in + (size_t)(r0 + i) * a.ld_in;
-      k = row[a.k_at + kv * N + n];
-      q = row[a.q_at + kv * N + n];
-      if (a.decay_mode == DECAY_CHANNEL) {
-        g = la_decay(a_log, decay_raw[(size_t)(r0 + i) * a.ld_decay + h * N + n] +
-                                a.dt_bias[h * N + n]);
-      } else if (a.decay_mode == DECAY_HEAD) {
-        g = la_decay(a_log, raw[(size_t)(r0 + i) * a.ld_raw + a.decay_at + h] + a.dt_bias[h]);
-      } else {
-        g = a.fixed[h];
+  const float rate = a.decay_mode == DECAY_FIXED ? 0.f : -expf(a.a_log[h]);
+  if (tid < LA_C * LA_C) {
+    A[tid / LA_C][tid % LA_C] = 0.f;
+    B[tid / LA_C][tid % LA_C] = 0.f;
+  }
+  // a warp per row: q and k (rotated, of unit length, scaled), the decays, beta
+  for (int i = warp; i < LA_C; i += LA_THREADS / 32) {
+    const bool row = i < count;
+    const float* src = in + (size_t)(r0 + i) * a.ld_in;
+    float k[NREG], q[NREG], g[NREG];
+    float shared_g = 1.f;
+    if (!CHANNEL && row) {
+      shared_g = a.decay_mode == DECAY_FIXED
+                     ? a.fixed[h]
+                     : la_decay(rate, raw[(size_t)(r0 + i) * a.ld_raw + a.decay_at + h] +
+                                          a.dt_bias[h]);
+    }
+#pragma unroll
+    for (int m = 0; m < NREG; ++m) {
+      const int n = lane + 32 * m;
+      const bool live = row && n < N;
+      k[m] = live ? src[a.k_at + kv * N + n] : 0.f;
+      q[m] = live ? src[a.q_at + kv * N + n] : 0.f;
+      g[m] = shared_g;
+      if (CHANNEL) {
+        g[m] = live ? la_decay(rate, decay_raw[(size_t)(r0 + i) * a.ld_decay + h * N + n] +
+                                         a.dt_bias[h * N + n])
+                    : 1.f;
       }
     }
-    k_s[idx] = k;
-    q_s[idx] = q;
-    g_s[idx] = g;
-  }
-  if (tid < LA_C) {
-    beta_s[tid] = (a.delta && tid < count)
-                      ? la_sigmoid(raw[(size_t)(r0 + tid) * a.ld_raw + a.beta_at + h]) : 0.f;
-  }
-  __syncthreads();
-  const int pairs = a.rot_dims / 2;
-  if (pairs > 0) {
-    for (int idx = tid; idx < count * pairs; idx += LA_THREADS) {
-      const int i = idx / pairs, pair = idx - i * pairs;
-      int x, y;
-      rope_members(pair, a.rot_dims, a.rot_layout, x, y);
-      float s, c;
-      la_sincos(a.positions[r0 + i], a.freq[pair], s, c);
-      float* kr = k_s + i * N;
-      float* qr = q_s + i * N;
-      const float ku = kr[x], kw = kr[y], qu = qr[x], qw = qr[y];
-      kr[x] = ku * c - kw * s;
-      kr[y] = kw * c + ku * s;
-      qr[x] = qu * c - qw * s;
-      qr[y] = qw * c + qu * s;
+    if (lane == 0) {
+      beta_s[i] = (a.delta && row)
+                      ? la_sigmoid(raw[(size_t)(r0 + i) * a.ld_raw + a.beta_at + h]) : 0.f;
     }
-    __syncthreads();
-  }
-  for (int i = warp; i < LA_C; i += LA_THREADS / 32) {  // lengths and scales, a warp per row
+    float* kr = k_s + i * NS;
+    float* qr = q_s + i * NS;
+    if (a.rot_dims > 0) {
+#pragma unroll
+      for (int m = 0; m < NREG; ++m) {
+        const int n = lane + 32 * m;
+        if (n < N) {
+          kr[n] = k[m];
+          qr[n] = q[m];
+        }
+      }
+      __syncwarp();
+      if (row) {
+        for (int pair = lane; pair < a.rot_dims / 2; pair += 32) {
+          int x, y;
+          rope_members(pair, a.rot_dims, a.rot_layout, x, y);
+          float s, c;
+          la_sincos(a.positions[r0 + i], a.freq[pair], s, c);
+          const float ku = kr[x], kw = kr[y], qu = qr[x], qw = qr[y];
+          kr[x] = ku * c - kw * s;
+          kr[y] = kw * c + ku * s;
+          qr[x] = qu * c - qw * s;
+          qr[y] = qw * c + qu * s;
+        }
+      }
+      __syncwarp();
+#pragma unroll
+      for (int m = 0; m < NREG; ++m) {
+        const int n = lane + 32 * m;
+        k[m] = n < N ? kr[n] : 0.f;
+        q[m] = n < N ? qr[n] : 0.f;
+      }
+    }
     float kf = a.k_scale, qf = a.q_scale;
     if (a.unit) {
       float kk = 0.f, qq = 0.f;
-      for (int n = lane; n < N; n += 32) {
-        kk = fmaf(k_s[i * N + n], k_s[i * N + n], kk);
-        qq = fmaf(q_s[i * N + n], q_s[i * N + n], qq);
+#pragma unroll
+      for (int m = 0; m < NREG; ++m) {
+        kk = fmaf(k[m], k[m], kk);
+        qq = fmaf(q[m], q[m], qq);
       }
       kf /= sqrtf(warp_sum(kk) + a.unit_eps);
       qf /= sqrtf(warp_sum(qq) + a.unit_eps);
     }
-    for (int n = lane; n < N; n += 32) {
-      k_s[i * N + n] *= kf;
-      q_s[i * N + n] *= qf;
+#pragma unroll
+    for (int m = 0; m < NREG; ++m) {
+      const int n = lane + 32 * m;
+      if (n < NS) {
+        kr[n] = k[m] * kf;
+        qr[n] = q[m] * qf;
+        g_s[i * NS + n] = g[m];
+      }
     }
   }
   __syncthreads();
@@ -264,85 +316,105 @@ la_prepare_kernel(const LinearArgs a) {
   float* kh_out = m_out + 2 * LA_C * N;
   float* g_out = kh_out + LA_C * N;
   float* r_out = g_out + la_pad4(N);
-  // A, B and D_(C-1) k: a warp takes columns j and C - 1 - j (together C + 1 rows of work)
-  for (int half = 0; half < 2; ++half) {
-    const int j = half ? LA_C - 1 - warp : warp;
-    float d[NREG];  // D_ij k_j, this lane's channels
+  {
+    // A, B and D_(C-1) k: warp w takes columns w and C - 1 - w, half a warp each, four
+    // neighbouring channels a lane at a time
+    constexpr int M = (NREG + 1) / 2;  // pieces of 16 lanes x 4 channels
+    const int half = lane >> 4, l = lane & 15, j = half ? LA_C - 1 - warp : warp;
+    float4 d[M];  // D_ij k_j (CHANNEL), else k_j, whose decays are one factor `dd`
+    float dd = 1.f;
 #pragma unroll
-    for (int m = 0; m < NREG; ++m) {
-      const int n = lane + 32 * m;
-      d[m] = n < N ? k_s[j * N + n] : 0.f;
+    for (int m = 0; m < M; ++m) {
+      const int n = 4 * (l + 16 * m);
+      d[m] = n < NS ? *reinterpret_cast<const float4*>(k_s + j * NS + n)
+                    : make_float4(0.f, 0.f, 0.f, 0.f);
     }
-    for (int i = j; i < LA_C; ++i) {
+    for (int i = warp; i < LA_C; ++i) {  // (warp: the smaller of the two columns)
       float sa = 0.f, sb = 0.f;
+      if (!CHANNEL && i > j) dd *= g_s[i * NS];
 #pragma unroll
-      for (int m = 0; m < NREG; ++m) {
-        const int n = lane + 32 * m;
-        if (n < N) {
-          if (i > j) d[m] *= g_s[i * N + n];
-          sa = fmaf(k_s[i * N + n], d[m], sa);
-          sb = fmaf(q_s[i * N + n], d[m], sb);
+      for (int m = 0; m < M; ++m) {
+        const int n = 4 * (l + 16 * m);
+        if (n < NS) {
+          const float4 k = *reinterpret_cast<const float4*>(k_s + i * NS + n);
+          const float4 q = *reinterpret_cast<const float4*>(q_s + i * NS + n);
+          if (CHANNEL && i > j) {
+            const float4 g = *reinterpret_cast<const float4*>(g_s + i * NS + n);
+            d[m].x *= g.x;
+            d[m].y *= g.y;
+            d[m].z *= g.z;
+            d[m].w *= g.w;
+          }
+          sa = fmaf(k.x, d[m].x, fmaf(k.y, d[m].y, fmaf(k.z, d[m].z, fmaf(k.w, d[m].w, sa))));
+          sb = fmaf(q.x, d[m].x, fmaf(q.y, d[m].y, fmaf(q.z, d[m].z, fmaf(q.w, d[m].w, sb))));
         }
       }
-      sa = warp_sum(sa);
-      sb = warp_sum(sb);
-      if (lane == 0) {
-        A[i][j] = sa;
-        B[i][j] = sb;
+#pragma unroll
+      for (int o = 8; o > 0; o >>= 1) {
+        sa += __shfl_xor_sync(0xffffffffu, sa, o);
+        sb += __shfl_xor_sync(0xffffffffu, sb, o);
+      }
+      if (l == 0 && i >= j) {
+        A[i][j] = sa * dd;
+        B[i][j] = sb * dd;
       }
     }
 #pragma unroll
-    for (int m = 0; m < NREG; ++m) {
-      const int n = lane + 32 * m;
-      if (n < N) w_s[j * N + n] = d[m];
-    }
-  }
-  for (int n = tid; n < N; n += LA_THREADS) {  // G, Kt, Qt
-    float g = 1.f;
-    float kt[LA_C], qt[LA_C];
-#pragma unroll
-    for (int i = 0; i < LA_C; ++i) {
-      g *= g_s[i * N + n];
-      kt[i] = g * k_s[i * N + n];
-      qt[i] = g * q_s[i * N + n];
-    }
-    g_out[n] = g;
-    float4* to = reinterpret_cast<float4*>(m_out + (size_t)n * 2 * LA_C);
-#pragma unroll
-    for (int i = 0; i < LA_C / 4; ++i) {
-      to[i] = make_float4(kt[4 * i], kt[4 * i + 1], kt[4 * i + 2], kt[4 * i + 3]);
-      to[LA_C / 4 + i] = make_float4(qt[4 * i], qt[4 * i + 1], qt[4 * i + 2], qt[4 * i + 3]);
+    for (int m = 0; m < M; ++m) {
+      const int n = 4 * (l + 16 * m);
+      if (n < NS) {
+        *reinterpret_cast<float4*>(w_s + j * NS + n) =
+            make_float4(d[m].x * dd, d[m].y * dd, d[m].z * dd, d[m].w * dd);
+      }
     }
   }
   __syncthreads();
-  if (tid < LA_C) {  // column `tid` of T, from the top
-    float x[LA_C];
+  if (warp == 0) {
+    if (lane < LA_C) {  // column `lane` of T, from the top (x[m] is 0 above the diagonal)
+      float x[LA_C];
 #pragma unroll
-    for (int i = 0; i < LA_C; ++i) {
-      float s = i == tid ? 1.f : 0.f;
-      if (a.delta) {
+      for (int i = 0; i < LA_C; ++i) {
+        float s = i == lane ? 1.f : 0.f;
+        if (a.delta) {
 #pragma unroll
-        for (int m = 0; m < i; ++m) {
-          s = fmaf(m >= tid ? -A[i][m] : 0.f, x[m], s);
+          for (int m = 0; m < i; ++m) s = fmaf(-A[i][m], x[m], s);
+          s *= beta_s[i];
         }
-        s *= beta_s[i];
+        x[i] = s;
+        T[i][lane] = s;
       }
-      x[i] = s;
-      T[i][tid] = i >= tid ? s : 0.f;
+    }
+  } else {  // meanwhile Kt and Qt (four rows of a channel a thread) and G
+    for (int idx = tid - 32; idx < N * 8; idx += LA_THREADS - 32) {
+      const int n = idx >> 3, part = idx & 7, first = (part & 3) * 4;
+      const float* x = part < 4 ? k_s : q_s;
+      float g = 1.f;
+      for (int i = 0; i < first; ++i) g *= g_s[i * NS + n];
+      float v[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        g *= g_s[(first + i) * NS + n];
+        v[i] = g * x[(first + i) * NS + n];
+      }
+      *reinterpret_cast<float4*>(m_out + (size_t)n * 2 * LA_C + part * 4) =
+          make_float4(v[0], v[1], v[2], v[3]);
+      if (part == 3) g_out[n] = g;
     }
   }
   __syncthreads();
-  if (tid < LA_C * LA_C) {
+  if (tid < LA_C * LA_C) {  // (B and T are zero above the diagonal)
     const int i = tid / LA_C, j = tid % LA_C;
     float s = 0.f;
-    for (int m = j; m <= i; ++m) s = fmaf(B[i][m], T[m][j], s);
+#pragma unroll
+    for (int m = 0; m < LA_C; ++m) s = fmaf(B[i][m], T[m][j], s);
     r_out[tid] = s;
   }
   for (int idx = tid; idx < N * (LA_C / 4); idx += LA_THREADS) {
     const int n = idx / (LA_C / 4), j = idx % (LA_C / 4) * 4;
     float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
-    for (int i = j; i < LA_C; ++i) {
-      const float d = w_s[i * N + n];
+#pragma unroll
+    for (int i = 0; i < LA_C; ++i) {
+      const float d = w_s[i * NS + n];
       const float4 t = *reinterpret_cast<const float4*>(&T[i][j]);
       s.x = fmaf(t.x, d, s.x);
       s.y = fmaf(t.y, d, s.y);
@@ -660,7 +732,7 @@ la_decode_kernel(const LinearArgs a, int PT) {
     }
   }
   if (a.decay_mode == DECAY_HEAD) {
-    const float g = la_decay(a.a_log[h], row[a.decay_at + h] + a.dt_bias[h]);
+    const float g = la_decay(-expf(a.a_log[h]), row[a.decay_at + h] + a.dt_bias[h]);
     for (int n = tid; n < N; n += threads) g_s[n] = g;
   } else if (a.decay_mode == DECAY_FIXED) {
     for (int n = tid; n < N; n += threads) g_s[n] = a.fixed[h];
@@ -668,9 +740,9 @@ la_decode_kernel(const LinearArgs a, int PT) {
   const float beta = a.delta ? la_sigmoid(row[a.beta_at + h]) : 1.f;
   __syncthreads();
   if (a.decay_mode == DECAY_CHANNEL) {
-    const float a_log = a.a_log[h];
+    const float rate = -expf(a.a_log[h]);
     la_matvec((const T*)a.decay_up + (size_t)h * N * a.decay_rank, low_s, a.decay_rank, N,
-              [&](int n, float z) { g_s[n] = la_decay(a_log, z + a.dt_bias[h * N + n]); });
+              [&](int n, float z) { g_s[n] = la_decay(rate, z + a.dt_bias[h * N + n]); });
   }
   if (a.gate_rank > 0) {
     la_matvec((const T*)a.gate_up + (size_t)h * P * a.gate_rank, low_s + a.decay_rank,
@@ -848,17 +920,22 @@ AYK_API int ayk_linear_chunks(const ayk::LinearArgs* args, void* stream) {
     return AYK_TOO_LARGE;
   }
   cudaStream_t s = (cudaStream_t)stream;
-  const size_t smem = (size_t)4 * LA_C * a.N * sizeof(float);
+  const size_t smem = (size_t)4 * LA_C * la_pad4(a.N) * sizeof(float);
   int status;
-#define AYK_LA_PREPARE(NREG)                                                                     \
+#define AYK_LA_PREPARE_AS(NREG, CHANNEL)                                                         \
   {                                                                                              \
     static const bool allowed =                                                                  \
-        (cudaFuncSetAttribute(la_prepare_kernel<NREG>,                                           \
+        (cudaFuncSetAttribute(la_prepare_kernel<NREG, CHANNEL>,                                  \
                               cudaFuncAttributeMaxDynamicSharedMemorySize,                       \
                               4 * LA_C * 32 * NREG * (int)sizeof(float)), true);                 \
     (void)allowed;                                                                               \
-    status = launch_kernel(la_prepare_kernel<NREG>, dim3(a.chunks, a.heads), dim3(LA_THREADS),   \
-                           smem, s, 1, a);                                                       \
+    status = launch_kernel(la_prepare_kernel<NREG, CHANNEL>, dim3(a.chunks, a.heads),            \
+                           dim3(LA_THREADS), smem, s, 1, a);                                     \
+  }
+#define AYK_LA_PREPARE(NREG)                                                                     \
+  {                                                                                              \
+    if (a.decay_mode == DECAY_CHANNEL) AYK_LA_PREPARE_AS(NREG, true)                             \
+    else AYK_LA_PREPARE_AS(NREG, false)                                                          \
   }
   if (a.N <= 32) AYK_LA_PREPARE(1)
   else if (a.N <= 64) AYK_LA_PREPARE(2)
@@ -866,6 +943,7 @@ AYK_API int ayk_linear_chunks(const ayk::LinearArgs* args, void* stream) {
   else if (a.N <= 256) AYK_LA_PREPARE(8)
   else AYK_LA_PREPARE(16)
 #undef AYK_LA_PREPARE
+#undef AYK_LA_PREPARE_AS
   if (status != AYK_OK) return status;
   const int vec = ((uintptr_t)a.in % 16) == 0 && a.ld_in % 4 == 0 && a.v_at % 4 == 0 &&
                   a.P % 4 == 0;

@@ -2172,6 +2172,11 @@ def conv_ring(x: torch.Tensor, weight: torch.Tensor, state: torch.Tensor, out: t
     check(status, op)
 
 
+#: a layer's argument struct (a launch copies it): what does not change from step to step is
+#: checked and filled in once per shape and set of constants
+_linear_structs: dict[tuple, _LinearArgs] = {}
+
+
 def _linear_args(op: str, shape: LinearShape, state: torch.Tensor, state_slot: torch.Tensor,
                  positions: torch.Tensor, a_log: torch.Tensor | None,
                  dt_bias: torch.Tensor | None, fixed: torch.Tensor | None,
@@ -2179,6 +2184,26 @@ def _linear_args(op: str, shape: LinearShape, state: torch.Tensor, state_slot: t
     _need(op, "state", state, torch.float32, 2)
     _need(op, "state_slot", state_slot, torch.int32, 1)
     _need(op, "positions", positions, torch.int32, 1)
+    if state.shape[1] < shape.ring_at + shape.taps * shape.channels:
+        raise BackendError(f"{op}: the state is too small")
+    # (the shapes' own numbers are in the key: an address alone may be used again)
+    key = (shape, *(None if t is None else (t.data_ptr(), t.shape[0])
+                    for t in (a_log, dt_bias, fixed, freq)))
+    args = _linear_structs.get(key)
+    if args is None:
+        args = _new_linear_args(op, shape, a_log, dt_bias, fixed, freq)
+        if len(_linear_structs) > 4096:
+            _linear_structs.clear()
+        _linear_structs[key] = args
+    args.positions, args.state_slot = positions.data_ptr(), state_slot.data_ptr()
+    args.state, args.state_stride = state.data_ptr(), state.stride(0)
+    args.q_at, args.k_at, args.v_at = shape.q_at, shape.k_at, shape.v_at
+    return args
+
+
+def _new_linear_args(op: str, shape: LinearShape, a_log: torch.Tensor | None,
+                     dt_bias: torch.Tensor | None, fixed: torch.Tensor | None,
+                     freq: torch.Tensor | None) -> _LinearArgs:
     for name, tensor, size in (
             ("fixed", fixed, shape.heads if shape.decay == "fixed" else None),
             ("a_log", a_log, shape.heads if shape.decay != "fixed" else None),
@@ -2190,8 +2215,6 @@ def _linear_args(op: str, shape: LinearShape, state: torch.Tensor, state_slot: t
             _need(op, name, tensor, torch.float32, 1)
             if tensor.shape[0] != size:
                 raise BackendError(f"{op}: {name} must hold {size} entries")
-    if state.shape[1] < shape.ring_at + shape.taps * shape.channels:
-        raise BackendError(f"{op}: the state is too small")
     rot_dims = 0 if freq is None else 2 * freq.shape[0]
     if rot_dims:
         _need(op, "freq", freq, torch.float64, 1)
@@ -2200,9 +2223,6 @@ def _linear_args(op: str, shape: LinearShape, state: torch.Tensor, state_slot: t
     args = _LinearArgs()
     args.a_log, args.dt_bias, args.fixed = _address(a_log), _address(dt_bias), _address(fixed)
     args.freq = _address(freq if rot_dims else None)
-    args.positions, args.state_slot = _address(positions), _address(state_slot)
-    args.state, args.state_stride = _address(state), state.stride(0)
-    args.q_at, args.k_at, args.v_at = shape.q_at, shape.k_at, shape.v_at
     args.decay_at, args.beta_at, args.gate_at = shape.decay_at, shape.beta_at, shape.gate_at
     args.heads, args.kv_heads, args.N, args.P = (shape.heads, shape.kv_heads, shape.dim,
                                                  shape.columns)

@@ -1,10 +1,12 @@
-"""``bench.py --design mapuvik`` / ``gagotar`` / ``semadra`` / ``rizitar``: prefill and decode
-throughput of the design at sizes that resemble a real model's layers, beside GPT-2 of the same
+"""``bench.py --design mapuvik`` / ``gagotar`` / ``semadra`` / ``rizitar`` / ``senurax``: prefill and
+decode throughput of the design at sizes that resemble a real model's layers, beside GPT-2 of the same
 width, heads, feed-forward and number of layers (Gagotar also beside Mapuvik, the design whose
 kernels are closest to its own; Semadra beside Gagotar, whose experts and attention, and
 Mapuvik, whose latent attention are the like kernels; Rizitar beside Semadra, whose windowed
 attention, norms behind the sublayers, experts and token input, and Gagotar, whose scan over a
-matrix state are the like kernels), on one B200 with random bf16 weights.
+matrix state are the like kernels; Senurax beside Rizitar, whose delta rule, Semadra, whose
+attention and gated experts, and Gagotar, whose linear attention beside a softmax attention are
+the like kernels), on one B200 with random bf16 weights.
 
 For each size and model: one prompt step of 2,048 tokens (two prompts of 1,024) and one decode
 step of 8 requests at context 1,025, each timed on the device as a CUDA-graph replay of the
@@ -123,6 +125,35 @@ def rizitar_config(width: int, heads: int, ff: int, repeats: int, vocab: int) ->
             "embedding": {"scale": width ** 0.5}, "token_side": {"dim": 64}, "layers": layers}
 
 
+#: Senurax at the bench's sizes: four layers of which the middle two run twice, so that a step
+#: runs six; retention heads of 64 x 128 with a dense feed-forward, delta heads of 64 x 64 with
+#: the experts of the other configurations plus two identity experts, two of eighteen per row
+SENURAX_EXPERTS, SENURAX_TOP, SENURAX_IDENTITY = 16, 2, 2
+
+
+def senurax_config(width: int, heads: int, ff: int, repeats: int, vocab: int) -> dict:
+    head = width // heads
+    memory = max(1, width // 128)
+    retention = {"heads": memory, "dim": 64, "vdim": 128,
+                 "decay": [1.0 - 2.0 ** -(5 + i % 8) for i in range(memory)],
+                 "rot": {"dims": 64, "base": 10000.0}}
+    delta = {"heads": width // 64, "kv_heads": width // 64, "dim": 64, "vdim": 64, "conv": 4}
+    channel = {**delta, "decay_rank": 64, "gate_rank": 64}
+    left = {"heads": heads, "kv_heads": heads // 4, "dim": head, "vdim": head,
+            "scale": head ** -0.5,
+            "rot": {"dims": head, "base": 500000.0, "scaling": {"factor": 4.0}}}
+    dense = {"kind": "dense", "ff": ff}
+    moe = {"kind": "moe", "expert": {"ff": ff // 4},
+           "router": {"experts": SENURAX_EXPERTS, "top": SENURAX_TOP,
+                      "identity": SENURAX_IDENTITY, "scale": 1.5}}
+    middle = [{"type": "channel_delta", "mixer": channel, "mlp": moe},
+              {"type": "parallel", "mixer": {"left": left, "right": delta}, "mlp": moe}]
+    ends = {"type": "retention", "mixer": retention, "mlp": dense}
+    return {"architecture": "Senurax", "vocab": vocab, "width": width, "norm": {"eps": 1e-5},
+            "logit_softcap": 30.0, "loop": {"start": 1, "stop": 3, "times": repeats},
+            "layers": [ends, *middle, ends]}
+
+
 def gpt2_config(width: int, heads: int, ff: int, layers: int, vocab: int) -> dict:
     return {"architectures": ["GPT2LMHeadModel"], "n_layer": layers, "n_embd": width,
             "n_head": heads, "n_inner": ff, "vocab_size": vocab, "n_positions": 2 * LENGTH,
@@ -216,6 +247,79 @@ def _class_work(config: dict, rows: int, keys_per_row: float, decode: bool,
             add("moe_experts", 2.0 * rows * top * 3 * f * width,
                 min(E, rows * top) * 3 * f * width * 2 + rows * top * (width * 6 + f * 4))
             add("moe_join", 0.0, rows * width * (4 * top + 8))
+        product(config["vocab"], width, 4, wanted)
+        return work
+    if config["architecture"] == "Senurax":
+        loop = config["loop"]
+        layers = config["layers"]
+        order = [*layers[:loop["start"]], *(layers[loop["start"]:loop["stop"]] * loop["times"]),
+                 *layers[loop["stop"]:]]
+
+        def linear_attention(m: dict, decay: int, taps: int, channel: bool) -> None:
+            """A recurrence and what goes with it: ``decay`` raw decays a row."""
+            H, kv, N, P = m["heads"], m.get("kv_heads", m["heads"]), m["dim"], m["vdim"]
+            channels = 2 * kv * N + H * P
+            state = 2 * H * N * P * 4 * (rows if decode else PROMPTS)
+            if decode:  # one kernel: convolution, low-rank pairs, state, norm and gate
+                up = H * (N + P) * m["gate_rank"] * 2 if channel else 0
+                add("linear_attention_decode", 8.0 * rows * H * N * P,
+                    rows * (channels * 4 * (1 + taps) + H * P * 6) + state + up)
+                return
+            if taps:
+                add("conv_ring", 2.0 * rows * channels * taps, rows * channels * 8)
+            if channel:
+                for rank, n in ((m["decay_rank"], H * N), (m["gate_rank"], H * P)):
+                    add("cast_rows", 0.0, rows * rank * 6)
+                    product(n, rank, 4)
+            add("linear_attention_chunks", 8.0 * rows * H * N * P,
+                rows * (channels + decay + H * P) * 4 + state)
+            add("rms_norm", 0.0, rows * H * P * 10)
+
+        add("cast_rows", 0.0, rows * width * 6 * (1 + loop["times"]))
+        for _ in range(loop["times"]):
+            product(width, 2 * width, 4)
+        for layer in order:
+            m, mlp = layer["mixer"], layer["mlp"]
+            add("rms_norm", 0.0, 2 * rows * width * 6)
+            if layer["type"] == "retention":
+                H, N, P = m["heads"], m["dim"], m["vdim"]
+                product(2 * H * (N + P), width, 4)
+                linear_attention(m, 0, 0, False)
+                product(width, H * P, 4)
+            elif layer["type"] == "channel_delta":
+                H, kv, N, P = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+                product(2 * kv * N + H * P + m["decay_rank"] + m["gate_rank"] + H, width, 4)
+                linear_attention(m, H * N, m["conv"], True)
+                product(width, H * P, 4)
+            else:
+                a, r = m["left"], m["right"]
+                H, G, dim, vdim = a["heads"], a["kv_heads"], a["dim"], a["vdim"]
+                product(H * dim + G * (dim + vdim), width, 4)
+                add("gated_attention_prepare", 0.0, rows * (H * dim + G * (dim + vdim)) * 6)
+                reuse = 1 if decode else 64 / 8  # a tile of 64 rows shares its keys
+                add("gated_attention", 2.0 * rows * keys_per_row * H * (dim + vdim),
+                    rows * keys_per_row * G * (dim + vdim) * 2 / reuse
+                    + rows * H * (dim + vdim) * 2)
+                product(width, H * vdim, 4)
+                H, kv, N, P = r["heads"], r["kv_heads"], r["dim"], r["vdim"]
+                product(2 * kv * N + 2 * H * P + 2 * H, width, 4)
+                linear_attention(r, H, r["conv"], False)
+                product(width, H * P, 4)
+                add("norm_sum", 0.0, rows * width * 16)
+            if mlp["kind"] == "dense":
+                product(mlp["ff"], width)
+                product(width, mlp["ff"], 4)
+            else:
+                router = mlp["router"]
+                E, top, f = router["experts"], router["top"], mlp["expert"]["ff"]
+                outputs = E + router["identity"]
+                pairs = rows * top * E / outputs  # (identity experts have no products)
+                product(outputs, width, 4)
+                add("moe_route_scored", 0.0, rows * (outputs + 2 * top) * 4)
+                add("moe_experts", 2.0 * pairs * 3 * f * width,
+                    min(E, pairs) * 3 * f * width * 2 + pairs * (width * 6 + f * 4))
+                add("moe_join", 0.0, rows * width * (4 * top + 8))
+        add("rms_norm", 0.0, wanted * width * 6)
         product(config["vocab"], width, 4, wanted)
         return work
     if config["architecture"] == "Rizitar":
@@ -457,7 +561,9 @@ def _measure(config: dict, peak: dict) -> dict:
                 torch.cuda.synchronize()
             for klass, pairs in record.items():
                 name = klass
-                if klass == "attention_prefill":
+                if klass == "attention_prefill" and "gated_attention" in work:
+                    name = "gated_attention"
+                elif klass == "attention_prefill":
                     name = "pooled_attention" if "pooled_attention" in work else (
                         "latent_attention" if "latent_attention" in work else "attention")
                 elif klass == "latent_decode":
@@ -471,7 +577,8 @@ def _measure(config: dict, peak: dict) -> dict:
             seconds = max(entry["us"], 1e-3) * 1e-6
             by_flops = work[name]["flops"] / seconds / tflops
             by_bytes = work[name]["bytes"] / seconds / gbs
-            tensor = not decode and "prepare" not in name and (
+            tensor = not decode and "prepare" not in name and \
+                    not name.startswith("linear_attention") and (
                 name.startswith("linear") or "attention" in name
                 or name in ("head_linear", "moe_experts"))
             entry["frac"] = round(by_flops if tensor else by_bytes, 4)
@@ -527,20 +634,24 @@ def run(sizes: str | None = None, design: str = "mapuvik") -> dict:
     for name in picked:
         width, heads, ff, repeats = table[name]
         results[name] = {"layers": 3 * repeats, "width": width, "heads": heads, "ff": ff}
-        if design == "rizitar":
+        if design == "senurax":
+            results[name]["senurax"] = _measure(
+                senurax_config(width, heads, ff, repeats, 32000), peak)
+        if design in ("rizitar", "senurax"):
             results[name]["rizitar"] = _measure(
                 rizitar_config(width, heads, ff, repeats, 32000), peak)
-        if design in ("semadra", "rizitar"):
+        if design in ("semadra", "rizitar", "senurax"):
             results[name]["semadra"] = _measure(
                 semadra_config(width, heads, ff, repeats, 32000), peak)
-        if design in ("gagotar", "semadra", "rizitar"):
+        if design in ("gagotar", "semadra", "rizitar", "senurax"):
             results[name]["gagotar"] = _measure(
                 gagotar_config(width, heads, ff, 3 * repeats, 32000), peak)
-        if design != "rizitar":
+        if design not in ("rizitar", "senurax"):
             results[name]["mapuvik"] = _measure(
                 mapuvik_config(width, heads, ff, repeats, 32000), peak)
         results[name]["gpt2"] = _measure(gpt2_config(width, heads, ff, 3 * repeats, 32000), peak)
-    title = {"rizitar": "Rizitar beside Semadra, Gagotar and GPT-2",
+    title = {"senurax": "Senurax beside Rizitar, Semadra, Gagotar and GPT-2",
+             "rizitar": "Rizitar beside Semadra, Gagotar and GPT-2",
              "gagotar": "Gagotar beside Mapuvik and GPT-2",
              "semadra": "Semadra beside Gagotar, Mapuvik and GPT-2"}.get(
                  design, "Mapuvik beside GPT-2")
