@@ -658,6 +658,15 @@ __device__ __forceinline__ void la_matvec(const T* W, const float* x, int rank, 
   }
 }
 
+// `bytes` from p on towards L2, shared out over the CTA. (A prefetch reads nothing, so what the
+// kernel ahead may still be writing may be named ahead of the dependency wait.)
+__device__ __forceinline__ void la_prefetch(const void* p, size_t bytes) {
+  const char* at = reinterpret_cast<const char*>(p);
+  for (size_t o = (size_t)threadIdx.x * 128; o < bytes; o += (size_t)blockDim.x * 128) {
+    asm volatile("prefetch.global.L2 [%0];" ::"l"(at + o));
+  }
+}
+
 template <typename T, int RN>
 __global__ void __launch_bounds__(512)
 la_decode_kernel(const LinearArgs a, int PT) {
@@ -679,6 +688,18 @@ la_decode_kernel(const LinearArgs a, int PT) {
   T* dst = reinterpret_cast<T*>(a.gated) + (size_t)r * a.ld_gated + (size_t)h * P;
   const float* in = a.in;
   float* state = a.state;
+  if (slot >= 0) {
+    const float* own = state + (size_t)slot * a.state_stride;
+    la_prefetch(own + (size_t)h * N * P, (size_t)N * P * sizeof(float));
+    if (a.decay_rank > 0) {
+      la_prefetch((const T*)a.decay_up + (size_t)h * N * a.decay_rank,
+                  (size_t)N * a.decay_rank * sizeof(T));
+    }
+    if (a.gate_rank > 0) {
+      la_prefetch((const T*)a.gate_up + (size_t)h * P * a.gate_rank,
+                  (size_t)P * a.gate_rank * sizeof(T));
+    }
+  }
   pdl_wait_for(in, state);
   if (slot < 0) {  // a row of padding (a graph's bucket): no request, no state
     for (int p = tid; p < P; p += threads) stf(dst + p, 0.f);
@@ -710,10 +731,19 @@ la_decode_kernel(const LinearArgs a, int PT) {
       const float* w = a.conv_weight + (size_t)channel * taps;
       const float x = row[c];
       float acc = w[taps - 1] * x;
-      for (int l = 1; l < taps && l <= position; ++l) {
-        int at = now - l;
-        if (at < 0) at += taps;
-        acc = fmaf(w[taps - 1 - l], ring[(size_t)at * a.channels + channel], acc);
+      for (int l0 = 1; l0 < taps; l0 += 3) {  // three earlier inputs on their way at once
+        float u[3], f[3];
+#pragma unroll
+        for (int e = 0; e < 3; ++e) {
+          const int l = l0 + e;
+          int at = now - l;
+          if (at < 0) at += taps;
+          const bool live = l < taps && l <= position;
+          u[e] = live ? ring[(size_t)at * a.channels + channel] : 0.f;
+          f[e] = live ? w[taps - 1 - l] : 0.f;
+        }
+#pragma unroll
+        for (int e = 0; e < 3; ++e) acc = fmaf(f[e], u[e], acc);
       }
       (part == 0 ? q_s : (part == 1 ? k_s : v_s))[e] = la_silu(acc);
       if (part == 2 || h % per == 0) ring[(size_t)now * a.channels + channel] = x;
@@ -828,7 +858,7 @@ la_decode_kernel(const LinearArgs a, int PT) {
 
 template <typename T>
 int la_decode(const LinearArgs& a, int rows, cudaStream_t s) {
-  const int threads = a.N > 256 || a.N * a.P > 8192 ? 512 : 256;
+  const int threads = a.N > 256 || a.N * a.P > 4096 ? 512 : 256;
   int PT = 256;
   while (PT > 32 && (PT / 2 >= a.P || a.N > 32 * (threads / PT))) PT /= 2;
   const int entries = (a.N + threads / PT - 1) / (threads / PT);

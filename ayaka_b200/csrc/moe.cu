@@ -498,16 +498,69 @@ moe_tile_kernel(const T* __restrict__ a, int lda, const T* __restrict__ weight,
 
 // dst[row][c] (+)= scale[c] * sum_j share[row * top + j] * pair_out[row * top + j][c]; a pair whose
 // choice is `experts` or more takes hidden[row][c] instead (an identity expert; `hidden` and
-// `chosen` are null when there is none).
+// `chosen` are null when there is none). With `next_out` (one CTA per row) also next_out[row] =
+// v rsqrt(mean(v^2) + next_eps) (next_offset + next_weight), v the new dst[row]: the norm in front
+// of the next sublayer, which may be written where `hidden` was read (a row's CTA has read all of
+// it by then).
 template <typename T>
 __global__ void moe_join_kernel(const float* __restrict__ pair_out, int ld, const float* __restrict__ share,
-                                const int* __restrict__ chosen, const T* __restrict__ hidden,
-                                int ld_hidden, int experts, int top,
+                                const int* __restrict__ chosen, const T* hidden, int ld_hidden,
+                                int experts, int top,
                                 const float* __restrict__ scale, float* __restrict__ dst,
-                                int ld_dst, int width, int accumulate) {
+                                int ld_dst, int width, int accumulate,
+                                const float* __restrict__ next_weight, float next_offset,
+                                float next_eps, T* next_out, int ld_next) {
+  __shared__ float scratch[33];
   pdl_launch_dependents();
   const int row = blockIdx.x;
+  constexpr int KEEP = 8;  // entries of a row a thread keeps in registers
+  if (next_out != nullptr && width <= KEEP * (int)blockDim.x) {
+    float ws[KEEP], ds[KEEP], sum[KEEP];
+#pragma unroll
+    for (int i = 0; i < KEEP; ++i) {
+      const int c = threadIdx.x + i * blockDim.x;
+      ws[i] = c < width ? next_offset + next_weight[c] : 0.f;
+      sum[i] = 0.f;
+    }
+    pdl_wait_for(pair_out, share, chosen, hidden, dst);
+#pragma unroll
+    for (int i = 0; i < KEEP; ++i) {
+      const int c = threadIdx.x + i * blockDim.x;
+      ds[i] = accumulate && c < width ? dst[(size_t)row * ld_dst + c] : 0.f;
+    }
+    for (int j = 0; j < top; ++j) {
+      const size_t pair = (size_t)row * top + j;
+      const bool identity = hidden != nullptr && chosen[pair] >= experts;
+      const float weight = share[pair];
+#pragma unroll
+      for (int i = 0; i < KEEP; ++i) {
+        const int c = threadIdx.x + i * blockDim.x;
+        if (c < width) {
+          sum[i] = fmaf(weight, identity ? ldf(hidden + (size_t)row * ld_hidden + c)
+                                         : pair_out[pair * ld + c], sum[i]);
+        }
+      }
+    }
+    float s2 = 0.f;
+#pragma unroll
+    for (int i = 0; i < KEEP; ++i) {
+      const int c = threadIdx.x + i * blockDim.x;
+      if (c < width) {
+        ds[i] += scale != nullptr ? sum[i] * scale[c] : sum[i];
+        dst[(size_t)row * ld_dst + c] = ds[i];
+        s2 += ds[i] * ds[i];
+      }
+    }
+    const float inv = 1.f / sqrtf(block_sum(s2, scratch) / (float)width + next_eps);
+#pragma unroll
+    for (int i = 0; i < KEEP; ++i) {
+      const int c = threadIdx.x + i * blockDim.x;
+      if (c < width) stf(next_out + (size_t)row * ld_next + c, ds[i] * inv * ws[i]);
+    }
+    return;
+  }
   pdl_wait_for(pair_out, share, chosen, hidden, dst);
+  float s2 = 0.f;
   for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < width; c += gridDim.y * blockDim.x) {
     float sum = 0.f;
     for (int j = 0; j < top; ++j) {
@@ -518,7 +571,16 @@ __global__ void moe_join_kernel(const float* __restrict__ pair_out, int ld, cons
     }
     if (scale != nullptr) sum *= scale[c];
     float* to = dst + (size_t)row * ld_dst + c;
-    *to = accumulate ? *to + sum : sum;
+    const float v = accumulate ? *to + sum : sum;
+    *to = v;
+    s2 += v * v;
+  }
+  if (next_out != nullptr) {  // (a thread reads back what it wrote itself)
+    const float inv = 1.f / sqrtf(block_sum(s2, scratch) / (float)width + next_eps);
+    for (int c = threadIdx.x; c < width; c += blockDim.x) {
+      stf(next_out + (size_t)row * ld_next + c,
+          dst[(size_t)row * ld_dst + c] * inv * (next_offset + next_weight[c]));
+    }
   }
 }
 
@@ -643,18 +705,24 @@ AYK_API int ayk_moe_experts(const void* hidden, int ld_hidden, const void* w_in,
 }
 
 // `hidden` (type: 0 = float32, 1 = bfloat16) with `chosen`: choices from `experts` on are identity
-// experts; both null: there is none.
+// experts; both null: there is none. `next_out` (of the same type; null: none) with `next_weight`:
+// the following norm's output.
 AYK_API int ayk_moe_join(const float* pair_out, int ld, const float* share, const int* chosen,
                          const void* hidden, int ld_hidden, int experts, int type, int rows,
                          int top, const float* scale, float* dst, int ld_dst, int width,
-                         int accumulate, void* stream) {
+                         int accumulate, const float* next_weight, float next_offset,
+                         float next_eps, void* next_out, int ld_next, void* stream) {
   using namespace ayk;
   if (rows == 0) return AYK_OK;
   if (rows < 0 || top < 1 || width < 1 || pair_out == nullptr || share == nullptr ||
       dst == nullptr || ld < width || ld_dst < width) {
     return AYK_BAD_ARGUMENT;
   }
-  const int threads = 256, tiles = min(8, (width + threads - 1) / threads);
+  if (next_out != nullptr && (next_weight == nullptr || ld_next < width || !(next_eps > 0.f))) {
+    return AYK_BAD_ARGUMENT;
+  }
+  const int threads = next_out != nullptr && width >= 1024 ? 512 : 256;
+  const int tiles = next_out != nullptr ? 1 : min(8, (width + threads - 1) / threads);
   if ((hidden == nullptr) != (chosen == nullptr) || (hidden != nullptr && ld_hidden < width)) {
     return AYK_BAD_ARGUMENT;
   }
@@ -662,9 +730,11 @@ AYK_API int ayk_moe_join(const float* pair_out, int ld, const float* share, cons
     return launch_kernel(moe_join_kernel<__nv_bfloat16>, dim3(rows, tiles), dim3(threads), 0,
                          (cudaStream_t)stream, 1, pair_out, ld, share, chosen,
                          (const __nv_bfloat16*)hidden, ld_hidden, experts, top, scale, dst, ld_dst,
-                         width, accumulate);
+                         width, accumulate, next_weight, next_offset, next_eps,
+                         (__nv_bfloat16*)next_out, ld_next);
   }
   return launch_kernel(moe_join_kernel<float>, dim3(rows, tiles), dim3(threads), 0,
                        (cudaStream_t)stream, 1, pair_out, ld, share, chosen, (const float*)hidden,
-                       ld_hidden, experts, top, scale, dst, ld_dst, width, accumulate);
+                       ld_hidden, experts, top, scale, dst, ld_dst, width, accumulate, next_weight,
+                       next_offset, next_eps, (float*)next_out, ld_next);
 }

@@ -15,7 +15,8 @@
 //
 // norm_sum: several fp32 rows of the same width, each normalised over the whole width with a
 // weight of its own, are averaged, multiplied element by element by an optional scale and
-// added to (or written into) an fp32 row: the join of mixers that run side by side.
+// added to (or written into) an fp32 row: the join of mixers that run side by side; the norm in
+// front of the next sublayer may leave the same launch.
 // Everything in fp32, rounded once to the output type. Any width.
 #include "common.cuh"
 
@@ -25,6 +26,10 @@ enum GateMode : int { GATE_NONE = 0, GATE_SILU_BEFORE = 1, GATE_SIGMOID_AFTER = 
                       GATE_SILU_AFTER = 3 };
 
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-z)); }
+
+// Entries a thread may keep in registers: a row of up to RN_KEEP a thread is read once, with the
+// weights on their way before the kernel ahead has finished.
+constexpr int RN_KEEP = 8;
 
 template <typename TOut>
 __global__ void rms_norm_kernel(const float* __restrict__ x, int ld_x,
@@ -36,6 +41,35 @@ __global__ void rms_norm_kernel(const float* __restrict__ x, int ld_x,
   pdl_launch_dependents();
   const int r = blockIdx.x, g = blockIdx.y;
   const int row = rows != nullptr ? rows[r] : r;
+  if (gate_mode == GATE_NONE && weight_period == 0 && group_width <= RN_KEEP * (int)blockDim.x) {
+    float ws[RN_KEEP], xs[RN_KEEP];
+#pragma unroll
+    for (int i = 0; i < RN_KEEP; ++i) {
+      const int c = threadIdx.x + i * blockDim.x;
+      ws[i] = 1.f;
+      if (c < group_width && weight != nullptr) {
+        ws[i] = weight_offset + weight[(size_t)g * group_width + c];
+      }
+    }
+    pdl_wait_for(x);
+    const float* src = x + (size_t)row * ld_x + (size_t)g * group_width;
+    float s = 0.f;
+#pragma unroll
+    for (int i = 0; i < RN_KEEP; ++i) {
+      const int c = threadIdx.x + i * blockDim.x;
+      xs[i] = c < group_width ? src[c] : 0.f;
+    }
+#pragma unroll
+    for (int i = 0; i < RN_KEEP; ++i) s += xs[i] * xs[i];
+    const float inv = 1.f / sqrtf(block_sum(s, scratch) / (float)group_width + eps);
+    TOut* dst = out + (size_t)r * ld_out + (size_t)g * group_width;
+#pragma unroll
+    for (int i = 0; i < RN_KEEP; ++i) {
+      const int c = threadIdx.x + i * blockDim.x;
+      if (c < group_width) stf(dst + c, xs[i] * inv * ws[i]);
+    }
+    return;
+  }
   pdl_wait_for(x, gate);
   const float* src = x + (size_t)row * ld_x + (size_t)g * group_width;
   const float* gt = gate != nullptr ? gate + (size_t)row * ld_gate + (size_t)g * group_width
@@ -174,14 +208,76 @@ struct Branches {
   int ld[SUM_MAX_BRANCHES];
 };
 
-// dst[r][c] (+)= scale[c] * factor * sum_b x_b[r][c] * rsqrt(mean_c(x_b[r]^2) + eps) * w_b[c]
+// dst[r][c] (+)= scale[c] * factor * sum_b x_b[r][c] * rsqrt(mean_c(x_b[r]^2) + eps) * w_b[c]; with
+// `next_out` also next_out[r] = the root-mean-square norm of the new dst[r] (see norm_add_kernel)
+template <typename TOut>
 __global__ void norm_sum_kernel(Branches in, int count, float eps, float factor,
                                 const float* __restrict__ scale, float* __restrict__ dst,
-                                int ld_dst, int width, int accumulate) {
+                                int ld_dst, int width, int accumulate,
+                                const float* __restrict__ next_weight, float next_offset,
+                                float next_eps, TOut* __restrict__ next_out, int ld_next) {
+  __shared__ float next_scratch[33];
   __shared__ float scratch[SUM_MAX_BRANCHES][32];
   pdl_launch_dependents();
   const int r = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int warps = (blockDim.x + 31) >> 5;
+  if (count == 2 && width <= RN_KEEP * (int)blockDim.x) {  // two sides, rows in registers
+    float ws[2][RN_KEEP], xs[2][RN_KEEP], ds[RN_KEEP];
+#pragma unroll
+    for (int i = 0; i < RN_KEEP; ++i) {
+      const int c = threadIdx.x + i * blockDim.x;
+      const float f = c < width ? (scale != nullptr ? scale[c] * factor : factor) : 0.f;
+#pragma unroll
+      for (int b = 0; b < 2; ++b) ws[b][i] = c < width ? in.weight[b][c] * f : 0.f;
+    }
+    pdl_wait_for(dst, in.x[0], in.x[1]);
+    float s[2] = {0.f, 0.f};
+#pragma unroll
+    for (int i = 0; i < RN_KEEP; ++i) {
+      const int c = threadIdx.x + i * blockDim.x;
+#pragma unroll
+      for (int b = 0; b < 2; ++b) xs[b][i] = c < width ? in.x[b][(size_t)r * in.ld[b] + c] : 0.f;
+      ds[i] = accumulate && c < width ? dst[(size_t)r * ld_dst + c] : 0.f;
+    }
+#pragma unroll
+    for (int i = 0; i < RN_KEEP; ++i) {
+#pragma unroll
+      for (int b = 0; b < 2; ++b) s[b] += xs[b][i] * xs[b][i];
+    }
+#pragma unroll
+    for (int b = 0; b < 2; ++b) {
+      s[b] = warp_sum(s[b]);
+      if (lane == 0) scratch[b][warp] = s[b];
+    }
+    __syncthreads();
+    float inv[2];
+#pragma unroll
+    for (int b = 0; b < 2; ++b) {
+      float sum = 0.f;
+      for (int w = 0; w < warps; ++w) sum += scratch[b][w];
+      inv[b] = 1.f / sqrtf(sum / (float)width + eps);
+    }
+    float s2 = 0.f;
+#pragma unroll
+    for (int i = 0; i < RN_KEEP; ++i) {
+      const int c = threadIdx.x + i * blockDim.x;
+      if (c < width) {
+        ds[i] += xs[0][i] * inv[0] * ws[0][i] + xs[1][i] * inv[1] * ws[1][i];
+        dst[(size_t)r * ld_dst + c] = ds[i];
+        s2 += ds[i] * ds[i];
+      }
+    }
+    if (next_out == nullptr) return;
+    const float inv2 = 1.f / sqrtf(block_sum(s2, next_scratch) / (float)width + next_eps);
+#pragma unroll
+    for (int i = 0; i < RN_KEEP; ++i) {
+      const int c = threadIdx.x + i * blockDim.x;
+      if (c < width) {
+        stf(next_out + (size_t)r * ld_next + c, ds[i] * inv2 * (next_offset + next_weight[c]));
+      }
+    }
+    return;
+  }
   pdl_wait_for(dst);
   // the branches' sums of squares side by side, through one exchange
   float inv[SUM_MAX_BRANCHES];
@@ -209,6 +305,7 @@ __global__ void norm_sum_kernel(Branches in, int count, float eps, float factor,
     }
   }
   float* to = dst + (size_t)r * ld_dst;
+  float s2 = 0.f;
   for (int c = threadIdx.x; c < width; c += blockDim.x) {
     float sum = 0.f;
 #pragma unroll
@@ -217,7 +314,15 @@ __global__ void norm_sum_kernel(Branches in, int count, float eps, float factor,
     }
     sum *= factor;
     if (scale != nullptr) sum *= scale[c];
-    to[c] = accumulate ? to[c] + sum : sum;
+    const float v = accumulate ? to[c] + sum : sum;
+    to[c] = v;
+    s2 += v * v;
+  }
+  if (next_out != nullptr) {  // (a thread reads back what it wrote itself)
+    const float inv2 = 1.f / sqrtf(block_sum(s2, next_scratch) / (float)width + next_eps);
+    for (int c = threadIdx.x; c < width; c += blockDim.x) {
+      stf(next_out + (size_t)r * ld_next + c, to[c] * inv2 * (next_offset + next_weight[c]));
+    }
   }
 }
 
@@ -329,13 +434,19 @@ AYK_API int ayk_rms_norm(const float* x, int ld_x, const int* rows, const float*
 }
 
 // `count` rows x[b] (fp32, leading dimension ld[b]) with weights w[b]; `scale` may be null.
+// `next_out` (next_type: 0 = float32, 1 = bfloat16; null: none) with `next_weight`: the following
+// norm's output.
 AYK_API int ayk_norm_sum(const float* const* x, const int* ld, const float* const* weight,
                          int count, float eps, float factor, const float* scale, float* dst,
-                         int ld_dst, int n, int width, int accumulate, void* stream) {
+                         int ld_dst, int n, int width, int accumulate, const float* next_weight,
+                         float next_offset, float next_eps, void* next_out, int ld_next,
+                         int next_type, void* stream) {
   using namespace ayk;
   if (n == 0) return AYK_OK;
   if (n < 0 || width < 1 || count < 1 || x == nullptr || ld == nullptr || weight == nullptr ||
-      dst == nullptr || ld_dst < width || !(eps > 0.f)) {
+      dst == nullptr || ld_dst < width || !(eps > 0.f) ||
+      (next_out != nullptr && (next_weight == nullptr || ld_next < width ||
+                               !(next_eps > 0.f) || (next_type != 0 && next_type != 1)))) {
     return AYK_BAD_ARGUMENT;
   }
   if (count > SUM_MAX_BRANCHES) return AYK_TOO_LARGE;
@@ -347,8 +458,15 @@ AYK_API int ayk_norm_sum(const float* const* x, const int* ld, const float* cons
     in.ld[b] = ld[b];
   }
   const int threads = width >= 2048 ? 512 : (width >= 512 ? 256 : 128);
-  return launch_kernel(norm_sum_kernel, dim3(n), dim3(threads), 0, (cudaStream_t)stream, 1, in,
-                       count, eps, factor, scale, dst, ld_dst, width, accumulate);
+  if (next_out != nullptr && next_type == 1) {
+    return launch_kernel(norm_sum_kernel<__nv_bfloat16>, dim3(n), dim3(threads), 0,
+                         (cudaStream_t)stream, 1, in, count, eps, factor, scale, dst, ld_dst, width,
+                         accumulate, next_weight, next_offset, next_eps, (__nv_bfloat16*)next_out,
+                         ld_next);
+  }
+  return launch_kernel(norm_sum_kernel<float>, dim3(n), dim3(threads), 0, (cudaStream_t)stream, 1,
+                       in, count, eps, factor, scale, dst, ld_dst, width, accumulate, next_weight,
+                       next_offset, next_eps, (float*)next_out, ld_next);
 }
 
 AYK_API int ayk_scale_add(const float* x, int ld_x, const float* scale, float* dst, int ld_dst,

@@ -1339,11 +1339,15 @@ def talking_attention(qmix: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.
 
 def norm_sum(branches: list[torch.Tensor], weights: list[torch.Tensor], eps: float,
              dst: torch.Tensor, *, factor: float, scale: torch.Tensor | None = None,
-             accumulate: bool = True, rows: int) -> None:
+             accumulate: bool = True, rows: int, next_weight: torch.Tensor | None = None,
+             next_eps: float = 1e-6, next_offset: float = 0.0,
+             next_out: torch.Tensor | None = None) -> None:
     """``dst (+)= scale * factor * sum_b rms_norm(branches[b]) * weights[b]``: up to four
     float32 ``[N, width]`` results, each normalised over the whole width by its root mean
     square with its own weight, summed, multiplied element by element by ``scale`` (float32
-    ``[width]``, optional) and added to (``accumulate``) or written into float32 ``dst``."""
+    ``[width]``, optional) and added to (``accumulate``) or written into float32 ``dst``; with
+    ``next_out`` (float32 or bfloat16) the new ``dst`` also leaves normalised for the sublayer
+    that follows, as in :func:`norm_add`."""
     op = "norm_sum"
     if _left_out and op in _left_out:
         return
@@ -1360,6 +1364,7 @@ def norm_sum(branches: list[torch.Tensor], weights: list[torch.Tensor], eps: flo
         _need(op, "scale", scale, torch.float32, 1)
         if scale.shape[0] != width:
             raise BackendError(f"{op}: the scale does not match the width")
+    _need_next(op, next_weight, next_out, width, rows)
     count = len(branches)
     xs = (c_void_p * count)(*[b.data_ptr() for b in branches])
     ws = (c_void_p * count)(*[w.data_ptr() for w in weights])
@@ -1367,8 +1372,27 @@ def norm_sum(branches: list[torch.Tensor], weights: list[torch.Tensor], eps: flo
     status = library("rms_norm").ayk_norm_sum(
         xs, lds, ws, c_int(count), c_float(eps), c_float(factor), _ptr(scale), _ptr(dst),
         c_int(dst.stride(0)), c_int(rows), c_int(width), c_int(1 if accumulate else 0),
-        _stream())
+        *_next_args(next_weight, next_offset, next_eps, next_out),
+        c_int(0 if next_out is None else _TYPE[next_out.dtype]), _stream())
     check(status, op)
+
+
+def _need_next(op: str, weight: torch.Tensor | None, out: torch.Tensor | None, width: int,
+               rows: int) -> None:
+    """The following norm's weight and output fit rows of ``width`` (``out`` ``None``: none)."""
+    if out is None:
+        return
+    _need(op, "next_out", out, ndim=2)
+    _need(op, "next_weight", weight, torch.float32, 1)
+    if out.dtype not in _TYPE or out.shape[1] != width or rows > out.shape[0] or \
+            weight.shape[0] != width:
+        raise BackendError(f"{op}: the next norm's output does not match dst")
+
+
+def _next_args(weight: torch.Tensor | None, offset: float, eps: float,
+               out: torch.Tensor | None) -> tuple:
+    return (_ptr(weight if out is not None else None), c_float(offset), c_float(eps), _ptr(out),
+            c_int(0 if out is None else out.stride(0)))
 
 
 def scale_add(x: torch.Tensor, scale: torch.Tensor, dst: torch.Tensor, *, rows: int,
@@ -1493,11 +1517,14 @@ def moe_experts(hidden: torch.Tensor, w_in: torch.Tensor, w_out: torch.Tensor,
 def moe_join(pair_out: torch.Tensor, share: torch.Tensor, dst: torch.Tensor, *, top: int,
              scale: torch.Tensor | None = None, accumulate: bool = True, rows: int,
              chosen: torch.Tensor | None = None, hidden: torch.Tensor | None = None,
-             experts: int = 0) -> None:
+             experts: int = 0, next_weight: torch.Tensor | None = None, next_eps: float = 1e-6,
+             next_offset: float = 0.0, next_out: torch.Tensor | None = None) -> None:
     """``dst[row] (+)= scale * sum_j share[row * top + j] * pair_out[row * top + j]`` in
     float32, the choices in order; ``scale`` (float32 ``[width]``) is optional. With
     ``hidden`` (the experts' input) and ``chosen``, a choice of ``experts`` or more is an
-    identity expert: ``hidden[row]`` stands for its ``pair_out``."""
+    identity expert: ``hidden[row]`` stands for its ``pair_out``. With ``next_out`` (``hidden``'s
+    type; it may be ``hidden`` itself) the new ``dst`` also leaves normalised for the sublayer
+    that follows, as in :func:`norm_add`."""
     op = "moe_join"
     if _left_out and op in _left_out:
         return
@@ -1518,13 +1545,18 @@ def moe_join(pair_out: torch.Tensor, share: torch.Tensor, dst: torch.Tensor, *, 
         if hidden.dtype not in _TYPE or hidden.shape[1] != width or hidden.shape[0] < rows or \
                 chosen.shape[0] < rows * top or experts < 1:
             raise BackendError(f"{op}: the identity experts' input does not match")
+    _need_next(op, next_weight, next_out, width, rows)
+    typed = hidden if hidden is not None else next_out
+    if next_out is not None and typed.dtype != next_out.dtype:
+        raise BackendError(f"{op}: hidden and the next norm's output have one type")
     status = library("moe").ayk_moe_join(
         _ptr(pair_out), c_int(pair_out.stride(0)), _ptr(share),
         _ptr(chosen if hidden is not None else None), _ptr(hidden),
         c_int(0 if hidden is None else hidden.stride(0)), c_int(experts),
-        c_int(0 if hidden is None else _TYPE[hidden.dtype]), c_int(rows), c_int(top),
+        c_int(0 if typed is None else _TYPE[typed.dtype]), c_int(rows), c_int(top),
         _ptr(scale), _ptr(dst), c_int(dst.stride(0)), c_int(width),
-        c_int(1 if accumulate else 0), _stream())
+        c_int(1 if accumulate else 0),
+        *_next_args(next_weight, next_offset, next_eps, next_out), _stream())
     check(status, op)
 
 

@@ -32,7 +32,11 @@ class PreNormBlock(Block):
     of the model's width (``mixer_scale``, ``feed_forward_scale``) before the sum: a part that
     has ``forward_scaled(hidden, residual, step[, cache], scale)`` applies the vector in its
     own last kernel; any other part writes into a scratch row that one more kernel scales and
-    adds."""
+    adds.
+
+    A half whose last kernel holds whole rows of the new stream (a part with
+    ``applies_next_norm``) also applies the norm in front of the next sublayer: the
+    feed-forward's, or the next layer's when the model names it (see SandwichNormBlock)."""
 
     def __init__(self, spec: LayerSpec, ctx: BuildContext, position: Part | None) -> None:
         super().__init__(ctx)
@@ -72,46 +76,73 @@ class PreNormBlock(Block):
     def forward(self, residual: torch.Tensor, step: StepContext, cache: LayerCache) -> None:
         n = step.num_rows
         hidden = step.workspace.buffer("block.normed", self.width, self.ctx.dtype)
-        if self.mixer_scale is not None:
-            self._forward_scaled(hidden, residual, step, cache)
-            return
+        # the norm of the layer that follows, and whether this layer's own has been applied by
+        # the launch that last updated the stream (see SandwichNormBlock)
+        following = step.extra.pop("block.next_norm", None)
+        if not (_can_follow(following) and following.width == self.width):
+            following = None
+        ready = step.extra.pop("block.normed_by", None) is self.mixer_norm
+        ff_norm = self.feed_forward_norm
         # a part that can apply the norm itself gets the residual and the norm part
-        if hasattr(self.mixer, "forward_normed") and _plain_norm(self.mixer_norm):
+        if self.mixer_scale is None and hasattr(self.mixer, "forward_normed") and \
+                _plain_norm(self.mixer_norm):
             self.mixer.forward_normed(self.mixer_norm, residual, step, cache)  # type: ignore
+            ready = False
         else:
-            self.mixer_norm.forward(residual, hidden, count=n)  # type: ignore[attr-defined]
-            self.mixer.forward(hidden, residual, step, cache)  # type: ignore[attr-defined]
-        if self.feed_forward_norm is None:
+            if not ready:
+                self.mixer_norm.forward(residual, hidden, count=n)  # type: ignore[attr-defined]
+            ready = self._mix(hidden, residual, step, cache,
+                              following if ff_norm is None else ff_norm)
+        if ff_norm is None:
+            if ready:
+                step.extra["block.normed_by"] = following
             return
-        if hasattr(self.feed_forward, "forward_normed") and _plain_norm(self.feed_forward_norm):
-            self.feed_forward.forward_normed(  # type: ignore[attr-defined]
-                self.feed_forward_norm, residual, step)
-        else:
-            self.feed_forward_norm.forward(residual, hidden, count=n)  # type: ignore
-            self.feed_forward.forward(hidden, residual, step)  # type: ignore[attr-defined]
+        if self.feed_forward_scale is None and hasattr(self.feed_forward, "forward_normed") and \
+                _plain_norm(ff_norm):
+            self.feed_forward.forward_normed(ff_norm, residual, step)  # type: ignore
+            return
+        if not ready:
+            ff_norm.forward(residual, hidden, count=n)  # type: ignore[attr-defined]
+        if self._feed(hidden, residual, step, following):
+            step.extra["block.normed_by"] = following
 
-
-    def _forward_scaled(self, hidden: torch.Tensor, residual: torch.Tensor, step: StepContext,
-                        cache: LayerCache) -> None:
-        n = step.num_rows
-        self.mixer_norm.forward(residual, hidden, count=n)  # type: ignore[attr-defined]
-        if hasattr(self.mixer, "forward_scaled"):
+    def _mix(self, hidden: torch.Tensor, residual: torch.Tensor, step: StepContext,
+             cache: LayerCache, then: object) -> bool:
+        """The mixer's half; True if its last kernel also left ``then(residual)`` in ``hidden``."""
+        then = then if hasattr(then, "as_next") and \
+            getattr(self.mixer, "applies_next_norm", False) else None
+        if then is not None:
+            self.mixer.forward_scaled(hidden, residual, step, cache,  # type: ignore
+                                      self.mixer_scale, then=then, then_out=hidden)
+        elif self.mixer_scale is None:
+            self.mixer.forward(hidden, residual, step, cache)  # type: ignore[attr-defined]
+        elif hasattr(self.mixer, "forward_scaled"):
             self.mixer.forward_scaled(hidden, residual, step, cache,  # type: ignore
                                       self.mixer_scale)
         else:
             branch = self._empty_branch(step)
             self.mixer.forward(hidden, branch, step, cache)  # type: ignore[attr-defined]
-            ops.scale_add(branch, self.mixer_scale, residual, rows=n)
-        if self.feed_forward_scale is None or self.feed_forward_norm is None:
-            return
-        self.feed_forward_norm.forward(residual, hidden, count=n)  # type: ignore
-        if hasattr(self.feed_forward, "forward_scaled"):
-            self.feed_forward.forward_scaled(hidden, residual, step,  # type: ignore
-                                             self.feed_forward_scale)
+            ops.scale_add(branch, self.mixer_scale, residual, rows=step.num_rows)
+        return then is not None
+
+    def _feed(self, hidden: torch.Tensor, residual: torch.Tensor, step: StepContext,
+              then: object) -> bool:
+        """The feed-forward's half; True if its last kernel left ``then(residual)`` in ``hidden``."""
+        scale = self.feed_forward_scale
+        then = then if hasattr(then, "as_next") and \
+            getattr(self.feed_forward, "applies_next_norm", False) else None
+        if then is not None:
+            self.feed_forward.forward_scaled(hidden, residual, step, scale,  # type: ignore
+                                             then=then, then_out=hidden)
+        elif scale is None:
+            self.feed_forward.forward(hidden, residual, step)  # type: ignore[attr-defined]
+        elif hasattr(self.feed_forward, "forward_scaled"):
+            self.feed_forward.forward_scaled(hidden, residual, step, scale)  # type: ignore
         else:
             branch = self._empty_branch(step)
             self.feed_forward.forward(hidden, branch, step)  # type: ignore[attr-defined]
-            ops.scale_add(branch, self.feed_forward_scale, residual, rows=n)
+            ops.scale_add(branch, scale, residual, rows=step.num_rows)
+        return then is not None
 
     def _empty_branch(self, step: StepContext) -> torch.Tensor:
         """A zeroed fp32 scratch row per row of the step (parts add into what they get)."""
@@ -149,7 +180,8 @@ class ParallelBlock(Block):
 def _can_follow(norm: object) -> bool:
     """Whether ``norm`` is a root-mean-square norm that ``ops.norm_add`` can apply on its way
     out (``weight``, ``offset``, ``eps`` and ``width``)."""
-    return all(hasattr(norm, name) for name in ("weight", "offset", "eps", "width"))
+    return norm is not None and all(hasattr(norm, name)
+                                    for name in ("weight", "offset", "eps", "width"))
 
 
 def _plain_norm(norm: Part | None) -> bool:

@@ -6,7 +6,7 @@ from __future__ import annotations
 import torch
 
 from ayaka_b200.kernels import ops
-from ayaka_b200.parts.base import BuildContext, build_part, register_part
+from ayaka_b200.parts.base import BuildContext, Part, build_part, register_part
 from ayaka_b200.parts.context import StepContext
 from ayaka_b200.parts.feed_forward import FeedForward
 from ayaka_b200.parts.spec import PartSpec
@@ -119,8 +119,15 @@ class MixtureOfExperts(FeedForward):
         """The same, written into ``out`` (fp32 ``[N, width]``) instead of added to it."""
         self.forward_scaled(hidden, out, step, None, accumulate=False)
 
+    @property
+    def applies_next_norm(self) -> bool:
+        """Whether ``forward_scaled`` takes ``then``: a root-mean-square norm that its last kernel
+        applies to the rows it has updated (not with a shared expert, which is added later)."""
+        return self.shared is None
+
     def forward_scaled(self, hidden: torch.Tensor, residual: torch.Tensor, step: StepContext,
-                       scale: torch.Tensor | None, accumulate: bool = True) -> None:
+                       scale: torch.Tensor | None, accumulate: bool = True,
+                       then: Part | None = None, then_out: torch.Tensor | None = None) -> None:
         n, work, top = step.num_rows, step.workspace, self.top
         # scratch for the largest step, so that its addresses never change
         most = work.max_rows
@@ -148,9 +155,10 @@ class MixtureOfExperts(FeedForward):
                         experts=self.experts, top=top, limit=self.limit, alpha=self.alpha,
                         shift=self.shift, sorted_pairs=sorted_pairs, tile_expert=tile_expert,
                         inner=inner, rows=n, single=self.single)
+        following = {} if then is None else then.as_next(then_out)  # type: ignore
         identity = dict(chosen=chosen, hidden=hidden, experts=self.experts) \
             if self.identity else {}
         ops.moe_join(pair_out, share, residual, top=top, scale=scale, accumulate=accumulate,
-                     rows=n, **identity)
+                     rows=n, **identity, **following)
         if self.shared is not None:
             self.shared.forward(hidden, residual, step)  # type: ignore[attr-defined]

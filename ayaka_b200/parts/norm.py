@@ -63,6 +63,12 @@ class RMSNorm(Part):
         ops.rms_norm(x, self.weight, self.eps, out, weight_offset=self.offset, rows=rows,
                      count=count)
 
+    def as_next(self, out: torch.Tensor) -> dict[str, object]:
+        """This norm as the norm in front of the next sublayer, for a kernel that applies it to
+        the rows it has just updated (``next_*`` of ``ops.norm_sum``, ``ops.moe_join``)."""
+        return dict(next_weight=self.weight, next_eps=self.eps, next_offset=self.offset,
+                    next_out=out)
+
     def add_normed(self, x: torch.Tensor, residual: torch.Tensor, *, factor: float, count: int,
                    copy: torch.Tensor | None = None, then: RMSNorm | None = None,
                    then_out: torch.Tensor | None = None) -> None:

@@ -60,8 +60,13 @@ class SideBySide(Mixer):
                 cache: LayerCache) -> None:
         self.forward_scaled(hidden, residual, step, cache, None)
 
+    #: ``forward_scaled`` takes ``then``: a root-mean-square norm that its last kernel applies
+    #: to the rows of the stream it has updated
+    applies_next_norm = True
+
     def forward_scaled(self, hidden: torch.Tensor, residual: torch.Tensor, step: StepContext,
-                       cache: LayerCache, scale: torch.Tensor | None) -> None:
+                       cache: LayerCache, scale: torch.Tensor | None,
+                       then: Part | None = None, then_out: torch.Tensor | None = None) -> None:
         n = step.num_rows
         branches = []
         for index, side in enumerate(self.sides):
@@ -72,8 +77,9 @@ class SideBySide(Mixer):
                 branch[:n].zero_()
                 side.forward(hidden, branch, step, cache)
             branches.append(branch)
+        following = {} if then is None else then.as_next(then_out)  # type: ignore
         ops.norm_sum(branches, self.weights, self.eps, residual, factor=1.0 / len(branches),
-                     scale=scale, accumulate=True, rows=n)
+                     scale=scale, accumulate=True, rows=n, **following)
 
 
 @register_part("mixer", "talking_attention")

@@ -215,6 +215,7 @@ def _class_work(config: dict, rows: int, keys_per_row: float, decode: bool,
         return work
     width = config["width"]
     if config["architecture"] == "Gagotar":
+        add("rms_norm", 0.0, rows * width * 6)  # (the others leave the sides' and experts' joins)
         for layer in config["layers"]:
             a, r, mlp = layer["mixer"]["left"], layer["mixer"]["right"], layer["mlp"]
             H, G, dim, vdim = a["heads"], a["kv_heads"], a["dim"], a["vdim"]
@@ -223,7 +224,6 @@ def _class_work(config: dict, rows: int, keys_per_row: float, decode: bool,
             # place of the context's last position in its block
             keys = (int(keys_per_row) - 1) % chunk + 1 if decode else \
                 sum(p % chunk + 1 for p in range(LENGTH)) / LENGTH
-            add("rms_norm", 0.0, 2 * rows * width * 6)
             product(H * dim + G * dim + G * vdim + H, width, 4)
             product(width, H * vdim, 4)
             add("talking_prepare", 2.0 * rows * H * H * dim,
@@ -240,13 +240,13 @@ def _class_work(config: dict, rows: int, keys_per_row: float, decode: bool,
                 rows * (3 * Hr * N + 2 * Hr * P) * 4 + (2 * Hr * N * P * 4) * (
                     rows if decode else 2))
             add("rms_norm", 0.0, rows * Hr * P * 10)
-            add("norm_sum", 0.0, rows * width * 16)
+            add("norm_sum", 0.0, rows * width * 18)
             E, top, f = mlp["router"]["experts"], mlp["router"]["top"], mlp["expert"]["ff"]
             product(E, width, 4)
             add("moe_route", 0.0, rows * (E + 2 * top) * 4)
             add("moe_experts", 2.0 * rows * top * 3 * f * width,
                 min(E, rows * top) * 3 * f * width * 2 + rows * top * (width * 6 + f * 4))
-            add("moe_join", 0.0, rows * width * (4 * top + 8))
+            add("moe_join", 0.0, rows * width * (4 * top + 10))
         product(config["vocab"], width, 4, wanted)
         return work
     if config["architecture"] == "Senurax":
@@ -278,9 +278,16 @@ def _class_work(config: dict, rows: int, keys_per_row: float, decode: bool,
         add("cast_rows", 0.0, rows * width * 6 * (1 + loop["times"]))
         for _ in range(loop["times"]):
             product(width, 2 * width, 4)
-        for layer in order:
+        # (a norm in front of a sublayer leaves the join of a mixer of two sides or of the
+        # experts, which then writes one more row in the compute type; it is a launch of its
+        # own behind the other kinds and ahead of a pass)
+        opens = {loop["start"] + p * (loop["stop"] - loop["start"]) for p in range(loop["times"])}
+        joined = False
+        for at, layer in enumerate(order):
             m, mlp = layer["mixer"], layer["mlp"]
-            add("rms_norm", 0.0, 2 * rows * width * 6)
+            launched = (0 if joined and at not in opens else 1) + (layer["type"] != "parallel")
+            add("rms_norm", 0.0, launched * rows * width * 6)
+            joined = mlp["kind"] == "moe"
             if layer["type"] == "retention":
                 H, N, P = m["heads"], m["dim"], m["vdim"]
                 product(2 * H * (N + P), width, 4)
@@ -305,7 +312,7 @@ def _class_work(config: dict, rows: int, keys_per_row: float, decode: bool,
                 product(2 * kv * N + 2 * H * P + 2 * H, width, 4)
                 linear_attention(r, H, r["conv"], False)
                 product(width, H * P, 4)
-                add("norm_sum", 0.0, rows * width * 16)
+                add("norm_sum", 0.0, rows * width * 18)
             if mlp["kind"] == "dense":
                 product(mlp["ff"], width)
                 product(width, mlp["ff"], 4)
@@ -319,6 +326,8 @@ def _class_work(config: dict, rows: int, keys_per_row: float, decode: bool,
                 add("moe_experts", 2.0 * pairs * 3 * f * width,
                     min(E, pairs) * 3 * f * width * 2 + pairs * (width * 6 + f * 4))
                 add("moe_join", 0.0, rows * width * (4 * top + 8))
+                if at + 1 < len(order) and at + 1 not in opens:
+                    add("moe_join", 0.0, rows * width * 2)
         add("rms_norm", 0.0, wanted * width * 6)
         product(config["vocab"], width, 4, wanted)
         return work
