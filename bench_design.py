@@ -570,11 +570,10 @@ def _measure(config: dict, peak: dict) -> dict:
                 torch.cuda.synchronize()
             for klass, pairs in record.items():
                 name = klass
-                if klass == "attention_prefill" and "gated_attention" in work:
-                    name = "gated_attention"
-                elif klass == "attention_prefill":
-                    name = "pooled_attention" if "pooled_attention" in work else (
-                        "latent_attention" if "latent_attention" in work else "attention")
+                if klass == "attention_prefill":
+                    name = next((kind for kind in ("pooled_attention", "latent_attention",
+                                                   "gated_attention") if kind in work),
+                                "attention")
                 elif klass == "latent_decode":
                     name = "latent_attention"
                 if name in work:
