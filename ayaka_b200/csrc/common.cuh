@@ -89,18 +89,17 @@ __device__ __forceinline__ float relu_squared(float x) {
   return y * y;
 }
 
+// (two tests on the common paths: each is paid in the epilogue of the few-rows products)
 __device__ __forceinline__ float activate(float x, int act) {
   if (act == ACT_GELU_TANH) return gelu_tanh(x);
-  if (act == ACT_GELU_ERF) return gelu_erf(x);
-  if (act == ACT_RELU_SQUARED) return relu_squared(x);
+  if (act >= ACT_GELU_ERF) return act == ACT_GELU_ERF ? gelu_erf(x) : relu_squared(x);
   return x;
 }
 
 // The same for a result that is stored as bfloat16.
 __device__ __forceinline__ float activate_to_bf16(float x, int act) {
   if (act == ACT_GELU_TANH) return gelu_tanh_fast(x);
-  if (act == ACT_GELU_ERF) return gelu_erf(x);
-  if (act == ACT_RELU_SQUARED) return relu_squared(x);
+  if (act >= ACT_GELU_ERF) return act == ACT_GELU_ERF ? gelu_erf(x) : relu_squared(x);
   return x;
 }
 
