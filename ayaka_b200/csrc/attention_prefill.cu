@@ -27,6 +27,12 @@
 // first, 64 at a time, then the window's keys. `sink` (one float per head): the softmax's
 // denominator also holds exp(sink[head]).
 //
+// -DAYK_SCORES chooses how scores become weights, at compile time, so that the softmax of the
+// other models carries nothing of it: 0 a softmax; 1 a softmax of scores from which `slope[head]`
+// times the key's distance has been taken; 2 sigmoid(score - slope * distance + score_bias[head])
+// per key, normalised over nothing: no maximum, no sum, the tile's weights go straight to the
+// second product.
+//
 // This kernel uses the legacy warp-level tensor path (not tcgen05): attention is ~5% of a
 // prefill step's FLOPs and this dataflow is proven; the matrix products that dominate run on
 // tcgen05 (gemm_tc.cu).
@@ -39,8 +45,15 @@
 #define AYK_VALUE_DIM AYK_HEAD_DIM
 #endif
 
+#ifndef AYK_SCORES
+#define AYK_SCORES 0
+#endif
+
 namespace ayk {
 
+constexpr int PF_SCORES = AYK_SCORES;
+constexpr bool PF_SLOPED = PF_SCORES != 0, PF_SIGMOID = PF_SCORES == 2;
+static_assert(PF_SCORES >= 0 && PF_SCORES <= 2, "scores");
 constexpr int PF_HD = AYK_HEAD_DIM;
 constexpr int PF_BM = 64;               // query rows per CTA
 constexpr int PF_BN = 64;               // keys per block
@@ -157,7 +170,8 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int ld_q,
                          const float* __restrict__ gate, int ld_gate, int pool, int pool_slots,
                          const __nv_bfloat16* __restrict__ k_pool,
                          const __nv_bfloat16* __restrict__ v_pool,
-                         const float* __restrict__ sink) {
+                         const float* __restrict__ sink, const float* __restrict__ slope,
+                         const float* __restrict__ score_bias) {
   extern __shared__ __align__(16) unsigned char pf_smem[];
   __nv_bfloat16* q_s = reinterpret_cast<__nv_bfloat16*>(pf_smem);
   __nv_bfloat16* k_s = q_s + PF_QTILE;      // two stages
@@ -247,6 +261,10 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int ld_q,
   float run_max[2] = {-INFINITY, -INFINITY}, run_sum[2] = {0.f, 0.f};
   const float scale2 = scale * 1.4426950408889634f;  // scores in units of log2
   const int row_a = pos0 + warp * 16 + (lane >> 2);  // position of this thread's first row
+  // what a position of distance takes off a score, and what every score gains (log2 units)
+  const float fall2 = PF_SLOPED && slope != nullptr ? slope[head] * 1.4426950408889634f : 0.f;
+  const float lift2 = PF_SIGMOID && score_bias != nullptr
+                          ? score_bias[head] * 1.4426950408889634f : 0.f;
   uint32_t q_frag[PF_HD / 16][4];
   bool q_loaded = false;
 
@@ -292,7 +310,9 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int ld_q,
     // mask, online softmax (rows row_a and row_a + 8). A block that lies wholly before the
     // warp's first row (and no window) has nothing to mask: only the scaling remains.
     const int key_base = block * PF_BN + (lane & 3) * 2;
-    const bool all_seen = window == 0 && block * PF_BN + PF_BN - 1 <= pos0 + warp * 16;
+    const bool all_seen =
+        !PF_SLOPED && window == 0 && block * PF_BN + PF_BN - 1 <= pos0 + warp * 16;
+    const float apart = PF_SLOPED ? (float)(row_a - key_base) : 0.f;
     float block_max[2] = {-INFINITY, -INFINITY};
     if (pooled && turn < kept_blocks) {
       // a turn of pooled rows: entry e is seen by the row at position p when
@@ -329,39 +349,53 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int ld_q,
           const int key = key_base + t * 8 + (e & 1);
           const int pos = row_a + (e >> 1) * 8;
           const bool seen = key <= pos && (window == 0 || key > pos - window || key < keep);
-          const float v = seen ? s[t][e] * scale2 : -INFINITY;
+          float scored = s[t][e] * scale2;
+          if (PF_SLOPED) {  // (the distance pos - key: whole numbers, exact in fp32)
+            scored = fmaf(-fall2, apart + (float)((e >> 1) * 8 - t * 8 - (e & 1)), scored);
+          }
+          if (PF_SIGMOID) scored += lift2;
+          const float v = seen ? scored : -INFINITY;
           s[t][e] = v;
-          block_max[e >> 1] = fmaxf(block_max[e >> 1], v);
+          if (!PF_SIGMOID) block_max[e >> 1] = fmaxf(block_max[e >> 1], v);
         }
       }
     }
-    float corr[2], ref[2];
+    if (PF_SIGMOID) {  // (a key out of sight: 2^inf, weight 0)
 #pragma unroll
-    for (int h = 0; h < 2; ++h) {
-      block_max[h] = fmaxf(block_max[h], __shfl_xor_sync(0xffffffffu, block_max[h], 1));
-      block_max[h] = fmaxf(block_max[h], __shfl_xor_sync(0xffffffffu, block_max[h], 2));
-      const float new_max = fmaxf(run_max[h], block_max[h]);
-      ref[h] = new_max == -INFINITY ? 0.f : new_max;
-      corr[h] = exp2f(run_max[h] - ref[h]);
-      run_max[h] = new_max;
-      run_sum[h] *= corr[h];
-    }
-    float part[2] = {0.f, 0.f};
+      for (int t = 0; t < PF_BN / 8; ++t) {
 #pragma unroll
-    for (int t = 0; t < PF_BN / 8; ++t) {
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const float p = exp2f(s[t][e] - ref[e >> 1]);
-        s[t][e] = p;
-        part[e >> 1] += p;
+        for (int e = 0; e < 4; ++e) s[t][e] = __fdividef(1.f, 1.f + exp2f(-s[t][e]));
       }
     }
-    run_sum[0] += part[0];
-    run_sum[1] += part[1];
+    float corr[2], ref[2];
+    if (!PF_SIGMOID) {
 #pragma unroll
-    for (int t = 0; t < PF_VD / 8; ++t) {
-      o[t][0] *= corr[0]; o[t][1] *= corr[0];
-      o[t][2] *= corr[1]; o[t][3] *= corr[1];
+      for (int h = 0; h < 2; ++h) {
+        block_max[h] = fmaxf(block_max[h], __shfl_xor_sync(0xffffffffu, block_max[h], 1));
+        block_max[h] = fmaxf(block_max[h], __shfl_xor_sync(0xffffffffu, block_max[h], 2));
+        const float new_max = fmaxf(run_max[h], block_max[h]);
+        ref[h] = new_max == -INFINITY ? 0.f : new_max;
+        corr[h] = exp2f(run_max[h] - ref[h]);
+        run_max[h] = new_max;
+        run_sum[h] *= corr[h];
+      }
+      float part[2] = {0.f, 0.f};
+#pragma unroll
+      for (int t = 0; t < PF_BN / 8; ++t) {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const float p = exp2f(s[t][e] - ref[e >> 1]);
+          s[t][e] = p;
+          part[e >> 1] += p;
+        }
+      }
+      run_sum[0] += part[0];
+      run_sum[1] += part[1];
+#pragma unroll
+      for (int t = 0; t < PF_VD / 8; ++t) {
+        o[t][0] *= corr[0]; o[t][1] *= corr[0];
+        o[t][2] *= corr[1]; o[t][3] *= corr[1];
+      }
     }
     // O += P V
 #pragma unroll
@@ -391,7 +425,7 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int ld_q,
     run_sum[h] += __shfl_xor_sync(0xffffffffu, run_sum[h], 1);
     run_sum[h] += __shfl_xor_sync(0xffffffffu, run_sum[h], 2);
   }
-  float inv0 = 1.f / run_sum[0], inv1 = 1.f / run_sum[1];
+  float inv0 = PF_SIGMOID ? 1.f : 1.f / run_sum[0], inv1 = PF_SIGMOID ? 1.f : 1.f / run_sum[1];
   if (sink != nullptr) {  // one more entry of the denominator, without a value
     const float sink2 = sink[head] * 1.4426950408889634f;
     float inv[2];
@@ -445,19 +479,25 @@ AYK_API int ayk_attention_prefill_value_dim() { return ayk::PF_VD; }
 // bfloat16 only. q/out rows are 16-byte aligned (ld multiples of 8 elements). `total_tiles`
 // = sum over requests of ceil(rows / 64), computed by the caller from its host copy of the
 // rows.
-// The same with pooled rows behind the window and a sink (see the head of this file); pool 0
-// and null pointers: none of them.
+// The same with pooled rows behind the window and a sink (see the head of this file; pool 0
+// and null pointers: none of them), and with slopes and biases of the scores (fp32, one per
+// head, may be null; only in a library compiled for them, see AYK_SCORES).
 AYK_API int ayk_attention_prefill_pooled(
     const void* q, int ld_q, const void* k_pages, const void* v_pages, const int* block_table,
     int table_stride, const int* row_start, const int* kv_len, void* out, int ld_out,
     int num_requests, int total_tiles, int num_heads, int num_kv_heads, int head_dim,
     int page_size, float scale, int window, int value_dim, int keep_first, const float* gate,
     int ld_gate, int pool, int pool_slots, const void* k_pool, const void* v_pool,
-    const float* sink, void* stream) {
+    const float* sink, const float* slope, const float* score_bias, void* stream) {
   using namespace ayk;
   if (num_requests == 0 || total_tiles == 0) return AYK_OK;
   if (head_dim != PF_HD || value_dim != PF_VD || keep_first < 0 ||
       (gate != nullptr && ld_gate < num_heads * PF_VD)) {
+    return AYK_BAD_ARGUMENT;
+  }
+  // (pooled rows stand at no one distance; a sink is an entry of a softmax)
+  if ((PF_SLOPED && pool > 0) || (PF_SIGMOID && sink != nullptr) ||
+      (!PF_SLOPED && slope != nullptr) || (!PF_SIGMOID && score_bias != nullptr)) {
     return AYK_BAD_ARGUMENT;
   }
   if (pool < 0 || (pool > 0 && window > 0 &&
@@ -503,7 +543,8 @@ AYK_API int ayk_attention_prefill_pooled(
                            kv_len, (__nv_bfloat16*)out, ld_out, num_requests, num_kv_heads,
                            num_heads / num_kv_heads, page_size, scale, window, total_tiles,
                            page_shift, keep_first, gate, ld_gate, pool, pool_slots,
-                           (const __nv_bfloat16*)k_pool, (const __nv_bfloat16*)v_pool, sink);
+                           (const __nv_bfloat16*)k_pool, (const __nv_bfloat16*)v_pool, sink,
+                           slope, score_bias);
     }
   }
   return launch_kernel(attention_prefill_kernel<false>, dim3(num_heads, total_tiles), dim3(128),
@@ -512,7 +553,8 @@ AYK_API int ayk_attention_prefill_pooled(
                        table_stride, row_start, kv_len, (__nv_bfloat16*)out, ld_out, num_requests,
                        num_kv_heads, num_heads / num_kv_heads, page_size, scale, window,
                        total_tiles, page_shift, keep_first, gate, ld_gate, pool, pool_slots,
-                           (const __nv_bfloat16*)k_pool, (const __nv_bfloat16*)v_pool, sink);
+                           (const __nv_bfloat16*)k_pool, (const __nv_bfloat16*)v_pool, sink,
+                           slope, score_bias);
 }
 
 AYK_API int ayk_attention_prefill(const void* q, int ld_q, const void* k_pages,
@@ -526,5 +568,5 @@ AYK_API int ayk_attention_prefill(const void* q, int ld_q, const void* k_pages,
                                       row_start, kv_len, out, ld_out, num_requests, total_tiles,
                                       num_heads, num_kv_heads, head_dim, page_size, scale, window,
                                       value_dim, keep_first, gate, ld_gate, 0, 0, nullptr,
-                                      nullptr, nullptr, stream);
+                                      nullptr, nullptr, nullptr, nullptr, stream);
 }

@@ -1,5 +1,6 @@
-// Softmax attention over paged keys and values with grouped heads, a value size of its own,
-// a sliding window that keeps the first tokens of the sequence in sight, and an output gate.
+// Attention over paged keys and values with grouped heads, a value size of its own, a sliding
+// window that keeps the first tokens of the sequence in sight, and an output gate. The weights
+// are a softmax over the visible keys or, key by key, a sigmoid that knows no other key.
 //
 // The query at position p of a request sees key j when j <= p and (p - j < window or
 // j < keep_first); window 0 means every earlier key. Kept tokens are ordinary keys at their
@@ -9,12 +10,16 @@
 // column 0 (H * dim), keys at k_off (G * dim), values at v_off (G * vdim): with norm weights
 // the whole query projection and the whole key projection are each divided by their root mean
 // square (one mean over all heads' entries, eps inside the root) and multiplied by a weight
-// per entry; with rotation frequencies the first rot_dims entries of every query and key head
+// per entry, or, with head_norm, every head by its own root mean square and multiplied by one
+// weight of dim entries that all heads share; with rotation frequencies the first rot_dims entries of every query and key head
 // are then rotated by the row's position; queries go to `q` in the compute type, the key and
 // value into the row's cache slot (pages [page][kv head][slot][dim or vdim]).
 //
-// attention: scores scale * (q . k), softmax and the weighted sum in fp32, the result times
-// sigmoid(gate) entry by entry when a gate (fp32, [row][H * vdim]) is given. The visible keys
+// attention: scores scale * (q . k), weights and the weighted sum in fp32, the result times
+// sigmoid(gate) entry by entry when a gate (fp32, [row][H * vdim]) is given. With `slope` (fp32,
+// [H]) the score of a key d positions back loses slope[h] * d (a kept key's true distance too).
+// SCORES_SIGMOID: a visible key's weight is sigmoid(score + score_bias[h]); nothing is
+// normalised over the keys, so there is no maximum and no sum to carry. The visible keys
 // are walked in a fixed order, first the kept ones that the window has left behind, then the
 // window, in tiles that start at the first visible key: what a row computes depends on its
 // position alone, not on the step's other rows.
@@ -30,6 +35,18 @@ namespace ayk {
 constexpr int GA_THREADS = 128;
 constexpr int GA_MAX_VALUE = 4;  // value entries per thread of the generic kernel (vdim <= 512)
 
+// how scores become weights: a softmax; a softmax of scores that fall with the distance; a
+// sigmoid per key (with or without slopes and biases)
+enum Scores : int { SCORES_SOFTMAX = 0, SCORES_SLOPED = 1, SCORES_SIGMOID = 2 };
+
+// the score of a key `apart` positions back, q . k already scaled
+template <int SCORES>
+__device__ __forceinline__ float placed_score(float scaled, float slope, float bias, int apart) {
+  if (SCORES == SCORES_SOFTMAX) return scaled;
+  return scaled - slope * (float)apart + bias;
+}
+__device__ __forceinline__ float sigmoid_of(float z) { return 1.f / (1.f + expf(-z)); }
+
 template <typename T>
 __global__ void __launch_bounds__(256)
 gated_prepare_kernel(const float* __restrict__ proj, int ld_proj, int k_off, int v_off,
@@ -37,7 +54,8 @@ gated_prepare_kernel(const float* __restrict__ proj, int ld_proj, int k_off, int
                      float eps, const int* __restrict__ slots, T* __restrict__ k_pages,
                      T* __restrict__ v_pages, int page_size, T* __restrict__ q, int ld_q, int H,
                      int G, int dim, int vdim, const int* __restrict__ positions,
-                     const double* __restrict__ freq, int rot_dims, int rot_layout) {
+                     const double* __restrict__ freq, int rot_dims, int rot_layout,
+                     int head_norm) {
   __shared__ float scratch[33];
   __shared__ float cos_s[ROPE_MAX_PAIRS], sin_s[ROPE_MAX_PAIRS];
   pdl_launch_dependents();
@@ -51,12 +69,12 @@ gated_prepare_kernel(const float* __restrict__ proj, int ld_proj, int k_off, int
   pdl_wait_for(proj);
   const float* src = proj + (size_t)row * ld_proj;
   float q_inv = 1.f, k_inv = 1.f;
-  if (q_weight != nullptr) {
+  if (q_weight != nullptr && !head_norm) {
     float s = 0.f;
     for (int i = tid; i < qn; i += blockDim.x) s += src[i] * src[i];
     q_inv = 1.f / sqrtf(block_sum(s, scratch) / (float)qn + eps);
   }
-  if (k_weight != nullptr) {
+  if (k_weight != nullptr && !head_norm) {
     float s = 0.f;
     for (int i = tid; i < kn; i += blockDim.x) s += src[k_off + i] * src[k_off + i];
     k_inv = 1.f / sqrtf(block_sum(s, scratch) / (float)kn + eps);
@@ -73,15 +91,31 @@ gated_prepare_kernel(const float* __restrict__ proj, int ld_proj, int k_off, int
     return second ? v * cos_s[pair] + o * sin_s[pair] : v * cos_s[pair] - o * sin_s[pair];
   };
   T* q_row = q + (size_t)row * ld_q;
-  for (int i = tid; i < qn; i += blockDim.x) {
-    stf(q_row + i, entry(src, q_weight, q_inv, i, i % dim));
-  }
-  if (slot < 0) return;
-  const size_t page = slot / page_size, at = slot % page_size;
-  for (int i = tid; i < kn; i += blockDim.x) {
-    const int g = i / dim, d = i % dim;
-    stf(k_pages + ((page * G + g) * page_size + at) * dim + d,
-        entry(src + k_off, k_weight, k_inv, i, d));
+  const size_t page = slot < 0 ? 0 : slot / page_size, at = slot < 0 ? 0 : slot % page_size;
+  if (head_norm) {  // a warp per head: its entries, its root mean square
+    const int lane = tid & 31;
+    for (int hh = tid >> 5; hh < H + (slot < 0 ? 0 : G); hh += blockDim.x >> 5) {
+      const bool query = hh < H;
+      const float* x = src + (query ? (size_t)hh * dim : k_off + (size_t)(hh - H) * dim);
+      const float* w = query ? q_weight : k_weight;
+      T* dst = query ? q_row + (size_t)hh * dim
+                     : k_pages + ((page * G + (hh - H)) * page_size + at) * dim;
+      float s = 0.f;
+      for (int d = lane; d < dim; d += 32) s += x[d] * x[d];
+      const float inv = w == nullptr ? 1.f : 1.f / sqrtf(warp_sum(s) / (float)dim + eps);
+      for (int d = lane; d < dim; d += 32) stf(dst + d, entry(x, w, inv, d, d));
+    }
+    if (slot < 0) return;
+  } else {
+    for (int i = tid; i < qn; i += blockDim.x) {
+      stf(q_row + i, entry(src, q_weight, q_inv, i, i % dim));
+    }
+    if (slot < 0) return;
+    for (int i = tid; i < kn; i += blockDim.x) {
+      const int g = i / dim, d = i % dim;
+      stf(k_pages + ((page * G + g) * page_size + at) * dim + d,
+          entry(src + k_off, k_weight, k_inv, i, d));
+    }
   }
   for (int i = tid; i < vn; i += blockDim.x) {
     const int g = i / vdim, d = i % vdim;
@@ -128,14 +162,15 @@ __device__ __forceinline__ float dot_row(const float* q, const __nv_bfloat16* k,
 // One CTA per (row, head). The visible keys, numbered 0 .. total - 1 (kept ones first), are
 // taken GA_THREADS at a time: a thread scores one key, the CTA keeps a running maximum and
 // sum, and thread c sums value entries c, c + GA_THREADS, ...
-template <typename T>
+template <typename T, int SCORES>
 __global__ void __launch_bounds__(GA_THREADS)
 gated_attention_kernel(const T* __restrict__ q, int ld_q, const T* __restrict__ k_pages,
                        const T* __restrict__ v_pages, const int* __restrict__ block_table,
                        int ld_table, const int* __restrict__ request_of_row,
                        const int* __restrict__ positions, const float* __restrict__ gate,
                        int ld_gate, T* __restrict__ out, int ld_out, int H, int G, int dim,
-                       int vdim, int page_size, float scale, int window, int keep_first) {
+                       int vdim, int page_size, float scale, int window, int keep_first,
+                       const float* __restrict__ slope, const float* __restrict__ score_bias) {
   extern __shared__ __align__(16) float ga_smem[];
   __shared__ float scratch[33];
   __shared__ float p_s[GA_THREADS];
@@ -155,6 +190,8 @@ gated_attention_kernel(const T* __restrict__ q, int ld_q, const T* __restrict__ 
   const int total = kept + position - lo + 1;
   const int kv = h / (H / G);
   const int* table = block_table + (size_t)b * ld_table;
+  const float fall = SCORES != SCORES_SOFTMAX && slope != nullptr ? slope[h] : 0.f;
+  const float lift = SCORES == SCORES_SIGMOID && score_bias != nullptr ? score_bias[h] : 0.f;
   pdl_wait_for(q, k_pages, v_pages, gate);
   for (int i = tid; i < dim; i += GA_THREADS) qv[i] = ldf(q + (size_t)row * ld_q + (size_t)h * dim + i);
   __syncthreads();
@@ -168,21 +205,28 @@ gated_attention_kernel(const T* __restrict__ q, int ld_q, const T* __restrict__ 
       const long long page = table[at / page_size];
       const long long base = (page * G + kv) * page_size + at % page_size;
       base_s[tid] = base;
-      score = dot_row(qv, k_pages + base * dim, dim) * scale;
+      score = placed_score<SCORES>(dot_row(qv, k_pages + base * dim, dim) * scale, fall, lift,
+                                   position - at);
     }
-    float best = warp_max(score);
-    __syncthreads();
-    if ((tid & 31) == 0) scratch[tid >> 5] = best;
-    __syncthreads();
-    best = scratch[0];
-    for (int w = 1; w < GA_THREADS / 32; ++w) best = fmaxf(best, scratch[w]);
-    const float m_new = fmaxf(m_run, best);  // (finite: a tile holds at least one key)
-    const float alpha = expf(m_run - m_new);
-    const float e = j < total ? expf(score - m_new) : 0.f;
-    p_s[tid] = e;
-    const float tile_sum = block_sum(e, scratch);  // (its barriers also publish p_s, base_s)
-    l_run = l_run * alpha + tile_sum;
-    m_run = m_new;
+    float alpha = 1.f;
+    if (SCORES == SCORES_SIGMOID) {
+      p_s[tid] = j < total ? sigmoid_of(score) : 0.f;
+      __syncthreads();
+    } else {
+      float best = warp_max(score);
+      __syncthreads();
+      if ((tid & 31) == 0) scratch[tid >> 5] = best;
+      __syncthreads();
+      best = scratch[0];
+      for (int w = 1; w < GA_THREADS / 32; ++w) best = fmaxf(best, scratch[w]);
+      const float m_new = fmaxf(m_run, best);  // (finite: a tile holds at least one key)
+      alpha = expf(m_run - m_new);
+      const float e = j < total ? expf(score - m_new) : 0.f;
+      p_s[tid] = e;
+      const float tile_sum = block_sum(e, scratch);  // (its barriers also publish p_s, base_s)
+      l_run = l_run * alpha + tile_sum;
+      m_run = m_new;
+    }
     const int n = min(GA_THREADS, total - j0);
 #pragma unroll
     for (int i = 0; i < GA_MAX_VALUE; ++i) {
@@ -201,7 +245,7 @@ gated_attention_kernel(const T* __restrict__ q, int ld_q, const T* __restrict__ 
   for (int i = 0; i < GA_MAX_VALUE; ++i) {
     const int c = tid + i * GA_THREADS;
     if (c < vdim) {
-      float v = acc[i] / l_run;
+      float v = SCORES == SCORES_SIGMOID ? acc[i] : acc[i] / l_run;
       if (gate != nullptr) v /= 1.f + expf(-gate[(size_t)row * ld_gate + (size_t)h * vdim + c]);
       stf(dst + c, v);
     }
@@ -241,7 +285,7 @@ template <> struct Piece<__nv_bfloat16> {
   }
 };
 
-template <typename T>
+template <typename T, int SCORES>
 __global__ void __launch_bounds__(GA_THREADS)
 gated_decode_kernel(const T* __restrict__ q, int ld_q, const T* __restrict__ k_pages,
                     const T* __restrict__ v_pages, const int* __restrict__ block_table,
@@ -249,7 +293,8 @@ gated_decode_kernel(const T* __restrict__ q, int ld_q, const T* __restrict__ k_p
                     const int* __restrict__ positions, const float* __restrict__ gate,
                     int ld_gate, float* __restrict__ partial, T* __restrict__ out, int ld_out,
                     int H, int G, int dim, int vdim, int page_size, float scale, int window,
-                    int keep_first) {
+                    int keep_first, const float* __restrict__ slope,
+                    const float* __restrict__ score_bias) {
   constexpr int VEC = Piece<T>::N;
   extern __shared__ __align__(16) float ga_smem[];
   __shared__ float scratch[33];
@@ -265,9 +310,11 @@ gated_decode_kernel(const T* __restrict__ q, int ld_q, const T* __restrict__ k_p
   const int b = request_of_row[row];
   T* dst = out + (size_t)row * ld_out + (size_t)h * vdim;
   float* part = partial + (((size_t)row * H + h) * shares + share) * (vdim + 2);
-  int first = 0, last = 0, lo = 0, kept = 0;
+  int first = 0, last = 0, lo = 0, kept = 0, position = 0;
+  const float fall = SCORES != SCORES_SOFTMAX && slope != nullptr ? slope[h] : 0.f;
+  const float lift = SCORES == SCORES_SIGMOID && score_bias != nullptr ? score_bias[h] : 0.f;
   if (b >= 0) {
-    const int position = positions[row];
+    position = positions[row];
     lo = window > 0 ? max(0, position - window + 1) : 0;
     kept = min(keep_first, lo);  // kept keys the window no longer covers
     const int total = kept + position - lo + 1;
@@ -300,21 +347,28 @@ gated_decode_kernel(const T* __restrict__ q, int ld_q, const T* __restrict__ k_p
       const long long page = table[at / page_size];
       const long long base = (page * G + kv) * page_size + at % page_size;
       base_s[tid] = base;
-      score = dot_row(qv, k_pages + base * dim, dim) * scale;
+      score = placed_score<SCORES>(dot_row(qv, k_pages + base * dim, dim) * scale, fall, lift,
+                                   position - at);
     }
-    float best = warp_max(score);
-    __syncthreads();
-    if ((tid & 31) == 0) scratch[tid >> 5] = best;
-    __syncthreads();
-    best = scratch[0];
-    for (int w = 1; w < GA_THREADS / 32; ++w) best = fmaxf(best, scratch[w]);
-    const float m_new = fmaxf(m_run, best);  // (finite: a tile holds at least one key)
-    const float alpha = expf(m_run - m_new);
-    const float e = j < last ? expf(score - m_new) : 0.f;
-    p_s[tid] = e;
-    const float tile_sum = block_sum(e, scratch);  // (its barriers also publish p_s, base_s)
-    l_run = l_run * alpha + tile_sum;
-    m_run = m_new;
+    float alpha = 1.f;
+    if (SCORES == SCORES_SIGMOID) {
+      p_s[tid] = j < last ? sigmoid_of(score) : 0.f;
+      __syncthreads();
+    } else {
+      float best = warp_max(score);
+      __syncthreads();
+      if ((tid & 31) == 0) scratch[tid >> 5] = best;
+      __syncthreads();
+      best = scratch[0];
+      for (int w = 1; w < GA_THREADS / 32; ++w) best = fmaxf(best, scratch[w]);
+      const float m_new = fmaxf(m_run, best);  // (finite: a tile holds at least one key)
+      alpha = expf(m_run - m_new);
+      const float e = j < last ? expf(score - m_new) : 0.f;
+      p_s[tid] = e;
+      const float tile_sum = block_sum(e, scratch);  // (its barriers also publish p_s, base_s)
+      l_run = l_run * alpha + tile_sum;
+      m_run = m_new;
+    }
     const int n = min(GA_THREADS, last - j0);
 #pragma unroll
     for (int i = 0; i < VEC; ++i) acc[i] *= alpha;
@@ -338,7 +392,7 @@ gated_decode_kernel(const T* __restrict__ q, int ld_q, const T* __restrict__ k_p
     float v = 0.f;
     for (int g = 0; g < groups; ++g) v += sums[g * vdim + c];
     if (shares == 1) {
-      v /= l_run;
+      if (SCORES != SCORES_SIGMOID) v /= l_run;
       if (gate != nullptr) v /= 1.f + expf(-gate[(size_t)row * ld_gate + (size_t)h * vdim + c]);
       stf(dst + c, v);
     } else {
@@ -351,8 +405,9 @@ gated_decode_kernel(const T* __restrict__ q, int ld_q, const T* __restrict__ k_p
   }
 }
 
-// One CTA per (row, head): the shares' results joined in the shares' order.
-template <typename T>
+// One CTA per (row, head): the shares' results joined in the shares' order (sums of sigmoid
+// weights are plain sums).
+template <typename T, bool NORMALISED>
 __global__ void __launch_bounds__(GA_THREADS)
 gated_merge_kernel(const float* __restrict__ partial, int shares,
                    const float* __restrict__ gate, int ld_gate, T* __restrict__ out, int ld_out,
@@ -362,54 +417,63 @@ gated_merge_kernel(const float* __restrict__ partial, int shares,
   pdl_wait_for(partial, gate);
   const float* part = partial + ((size_t)row * H + h) * shares * (vdim + 2);
   float m = -INFINITY;
-  for (int s = 0; s < shares; ++s) m = fmaxf(m, part[(size_t)s * (vdim + 2)]);
   float l = 0.f;
-  for (int s = 0; s < shares; ++s) {
-    const float ms = part[(size_t)s * (vdim + 2)];
-    if (ms > -INFINITY) l += part[(size_t)s * (vdim + 2) + 1] * expf(ms - m);
+  if (NORMALISED) {
+    for (int s = 0; s < shares; ++s) m = fmaxf(m, part[(size_t)s * (vdim + 2)]);
+    for (int s = 0; s < shares; ++s) {
+      const float ms = part[(size_t)s * (vdim + 2)];
+      if (ms > -INFINITY) l += part[(size_t)s * (vdim + 2) + 1] * expf(ms - m);
+    }
   }
   for (int c = threadIdx.x; c < vdim; c += GA_THREADS) {
     float v = 0.f;
-    for (int s = 0; s < shares; ++s) {
-      const float ms = part[(size_t)s * (vdim + 2)];
-      if (ms > -INFINITY) v += part[(size_t)s * (vdim + 2) + 2 + c] * expf(ms - m);
+    if (NORMALISED) {
+      for (int s = 0; s < shares; ++s) {
+        const float ms = part[(size_t)s * (vdim + 2)];
+        if (ms > -INFINITY) v += part[(size_t)s * (vdim + 2) + 2 + c] * expf(ms - m);
+      }
+      v = l > 0.f ? v / l : 0.f;  // (a row of padding has no keys)
+    } else {
+#pragma unroll 8
+      for (int s = 0; s < shares; ++s) v += part[(size_t)s * (vdim + 2) + 2 + c];
     }
-    v = l > 0.f ? v / l : 0.f;  // (a row of padding has no keys)
     if (gate != nullptr) v /= 1.f + expf(-gate[(size_t)row * ld_gate + (size_t)h * vdim + c]);
     stf(out + (size_t)row * ld_out + (size_t)h * vdim + c, v);
   }
 }
 
-template <typename T>
+template <typename T, int SCORES>
 int gated_decode(const void* q, int ld_q, const void* k_pages, const void* v_pages,
                  const int* block_table, int ld_table, const int* request_of_row,
                  const int* positions, const float* gate, int ld_gate, float* partial,
                  void* out, int ld_out, int rows, int H, int G, int dim, int vdim,
-                 int page_size, float scale, int window, int keep_first, int shares,
-                 cudaStream_t s) {
+                 int page_size, float scale, int window, int keep_first, const float* slope,
+                 const float* score_bias, int shares, cudaStream_t s) {
   const int columns = vdim / Piece<T>::N;
   const size_t smem = ((size_t)dim + (size_t)(GA_THREADS / columns) * vdim) * sizeof(float);
   int status = launch_kernel(
-      gated_decode_kernel<T>, dim3(shares, H, rows), dim3(GA_THREADS), smem, s, 1, (const T*)q,
-      ld_q, (const T*)k_pages, (const T*)v_pages, block_table, ld_table, request_of_row,
-      positions, gate, ld_gate, partial, (T*)out, ld_out, H, G, dim, vdim, page_size, scale,
-      window, keep_first);
+      gated_decode_kernel<T, SCORES>, dim3(shares, H, rows), dim3(GA_THREADS), smem, s, 1,
+      (const T*)q, ld_q, (const T*)k_pages, (const T*)v_pages, block_table, ld_table,
+      request_of_row, positions, gate, ld_gate, partial, (T*)out, ld_out, H, G, dim, vdim,
+      page_size, scale, window, keep_first, slope, score_bias);
   if (status != AYK_OK || shares == 1) return status;
-  return launch_kernel(gated_merge_kernel<T>, dim3(rows, H), dim3(GA_THREADS), 0, s, 1,
-                       (const float*)partial, shares, gate, ld_gate, (T*)out, ld_out, H, vdim);
+  return launch_kernel(gated_merge_kernel<T, SCORES != SCORES_SIGMOID>, dim3(rows, H),
+                       dim3(GA_THREADS), 0, s, 1, (const float*)partial, shares, gate, ld_gate,
+                       (T*)out, ld_out, H, vdim);
 }
 
-template <typename T>
+template <typename T, int SCORES>
 int gated_attention(const void* q, int ld_q, const void* k_pages, const void* v_pages,
                     const int* block_table, int ld_table, const int* request_of_row,
                     const int* positions, const float* gate, int ld_gate, void* out, int ld_out,
                     int rows, int H, int G, int dim, int vdim, int page_size, float scale,
-                    int window, int keep_first, cudaStream_t s) {
-  return launch_kernel(gated_attention_kernel<T>, dim3(rows, H), dim3(GA_THREADS),
+                    int window, int keep_first, const float* slope, const float* score_bias,
+                    cudaStream_t s) {
+  return launch_kernel(gated_attention_kernel<T, SCORES>, dim3(rows, H), dim3(GA_THREADS),
                        (size_t)dim * sizeof(float), s, 1, (const T*)q, ld_q, (const T*)k_pages,
                        (const T*)v_pages, block_table, ld_table, request_of_row, positions, gate,
                        ld_gate, (T*)out, ld_out, H, G, dim, vdim, page_size, scale, window,
-                       keep_first);
+                       keep_first, slope, score_bias);
 }
 
 }  // namespace ayk
@@ -418,12 +482,13 @@ AYK_API void ayk_set_pdl(int on) { ayk::pdl_enabled() = on; }
 
 // type: 0 = float32, 1 = bfloat16 (of q and the pages). Norm weights, slots and pages may be
 // null (no norm; nothing stored). rot_dims 0: no rotation (positions and freq may be null).
+// head_norm: the weights have dim entries and every head its own root mean square.
 AYK_API int ayk_gated_prepare(const float* proj, int ld_proj, int k_off, int v_off,
                               const float* q_weight, const float* k_weight, float eps,
                               const int* slots, void* k_pages, void* v_pages, int page_size,
                               void* q, int ld_q, int rows, int heads, int kv_heads, int dim,
                               int vdim, const int* positions, const double* freq, int rot_dims,
-                              int rot_layout, int type, void* stream) {
+                              int rot_layout, int head_norm, int type, void* stream) {
   using namespace ayk;
   if (rows == 0) return AYK_OK;
   if (rot_dims < 0 || rot_dims % 2 || rot_dims > dim || rot_dims > 2 * ROPE_MAX_PAIRS ||
@@ -442,19 +507,20 @@ AYK_API int ayk_gated_prepare(const float* proj, int ld_proj, int k_off, int v_o
     return launch_kernel(gated_prepare_kernel<float>, dim3(rows), dim3(256), 0, s, 1, proj,
                          ld_proj, k_off, v_off, q_weight, k_weight, eps, slots, (float*)k_pages,
                          (float*)v_pages, page_size, (float*)q, ld_q, heads, kv_heads, dim, vdim,
-                         positions, freq, rot_dims, rot_layout);
+                         positions, freq, rot_dims, rot_layout, head_norm);
   }
   if (type == 1) {
     return launch_kernel(gated_prepare_kernel<__nv_bfloat16>, dim3(rows), dim3(256), 0, s, 1,
                          proj, ld_proj, k_off, v_off, q_weight, k_weight, eps, slots,
                          (__nv_bfloat16*)k_pages, (__nv_bfloat16*)v_pages, page_size,
                          (__nv_bfloat16*)q, ld_q, heads, kv_heads, dim, vdim, positions, freq,
-                         rot_dims, rot_layout);
+                         rot_dims, rot_layout, head_norm);
   }
   return AYK_BAD_ARGUMENT;
 }
 
-// Steps of single rows. type as above. `partial`: float32 scratch of rows * heads * shares *
+// Steps of single rows. type as above; scores, slope, score_bias: how scores become weights (see
+// Scores; the vectors may be null). `partial`: float32 scratch of rows * heads * shares *
 // (vdim + 2) elements (not needed with one share). AYK_NOT_TAKEN, having run nothing, for
 // value rows that are not whole 16-byte pieces.
 AYK_API int ayk_gated_decode(const void* q, int ld_q, const void* k_pages, const void* v_pages,
@@ -462,7 +528,8 @@ AYK_API int ayk_gated_decode(const void* q, int ld_q, const void* k_pages, const
                              const int* positions, const float* gate, int ld_gate,
                              float* partial, void* out, int ld_out, int rows, int heads,
                              int kv_heads, int dim, int vdim, int page_size, float scale,
-                             int window, int keep_first, int shares, int type, void* stream) {
+                             int window, int keep_first, int scores, const float* slope,
+                             const float* score_bias, int shares, int type, void* stream) {
   using namespace ayk;
   if (rows == 0) return AYK_OK;
   if (rows < 0 || heads < 1 || kv_heads < 1 || heads % kv_heads || dim < 1 || vdim < 1 ||
@@ -470,7 +537,8 @@ AYK_API int ayk_gated_decode(const void* q, int ld_q, const void* k_pages, const
       k_pages == nullptr || v_pages == nullptr || block_table == nullptr ||
       request_of_row == nullptr || positions == nullptr || out == nullptr ||
       ld_q < heads * dim || ld_out < heads * vdim || (shares > 1 && partial == nullptr) ||
-      (gate != nullptr && ld_gate < heads * vdim) || (type != 0 && type != 1)) {
+      (gate != nullptr && ld_gate < heads * vdim) || (type != 0 && type != 1) ||
+      scores < SCORES_SOFTMAX || scores > SCORES_SIGMOID) {
     return AYK_BAD_ARGUMENT;
   }
   const int piece = type == 0 ? 4 : 8;
@@ -479,16 +547,20 @@ AYK_API int ayk_gated_decode(const void* q, int ld_q, const void* k_pages, const
     return AYK_NOT_TAKEN;
   }
   cudaStream_t s = (cudaStream_t)stream;
+#define AYK_GD(T, S)                                                                           \
+  return gated_decode<T, S>(q, ld_q, k_pages, v_pages, block_table, ld_table, request_of_row,  \
+                            positions, gate, ld_gate, partial, out, ld_out, rows, heads,       \
+                            kv_heads, dim, vdim, page_size, scale, window, keep_first, slope,  \
+                            score_bias, shares, s)
   if (type == 0) {
-    return gated_decode<float>(q, ld_q, k_pages, v_pages, block_table, ld_table,
-                               request_of_row, positions, gate, ld_gate, partial, out, ld_out,
-                               rows, heads, kv_heads, dim, vdim, page_size, scale, window,
-                               keep_first, shares, s);
+    if (scores == SCORES_SIGMOID) AYK_GD(float, SCORES_SIGMOID);
+    if (scores == SCORES_SLOPED) AYK_GD(float, SCORES_SLOPED);
+    AYK_GD(float, SCORES_SOFTMAX);
   }
-  return gated_decode<__nv_bfloat16>(q, ld_q, k_pages, v_pages, block_table, ld_table,
-                                     request_of_row, positions, gate, ld_gate, partial, out,
-                                     ld_out, rows, heads, kv_heads, dim, vdim, page_size, scale,
-                                     window, keep_first, shares, s);
+  if (scores == SCORES_SIGMOID) AYK_GD(__nv_bfloat16, SCORES_SIGMOID);
+  if (scores == SCORES_SLOPED) AYK_GD(__nv_bfloat16, SCORES_SLOPED);
+  AYK_GD(__nv_bfloat16, SCORES_SOFTMAX);
+#undef AYK_GD
 }
 
 // mode: 0 = the generic kernel; 1 = the tensor-core kernel where the sizes allow (bfloat16).
@@ -497,7 +569,8 @@ AYK_API int ayk_gated_attention(const void* q, int ld_q, const void* k_pages,
                                 const int* request_of_row, const int* positions,
                                 const float* gate, int ld_gate, void* out, int ld_out, int rows,
                                 int heads, int kv_heads, int dim, int vdim, int page_size,
-                                float scale, int window, int keep_first, int mode, int type,
+                                float scale, int window, int keep_first, int scores,
+                                const float* slope, const float* score_bias, int mode, int type,
                                 void* stream) {
   using namespace ayk;
   if (rows == 0) return AYK_OK;
@@ -505,23 +578,25 @@ AYK_API int ayk_gated_attention(const void* q, int ld_q, const void* k_pages,
       page_size < 1 || window < 0 || keep_first < 0 || q == nullptr || k_pages == nullptr ||
       v_pages == nullptr || block_table == nullptr || request_of_row == nullptr ||
       positions == nullptr || out == nullptr || ld_q < heads * dim || ld_out < heads * vdim ||
-      (gate != nullptr && ld_gate < heads * vdim)) {
+      (gate != nullptr && ld_gate < heads * vdim) || (type != 0 && type != 1) ||
+      scores < SCORES_SOFTMAX || scores > SCORES_SIGMOID) {
     return AYK_BAD_ARGUMENT;
   }
   if (vdim > GA_THREADS * GA_MAX_VALUE || dim > 8192) return AYK_TOO_LARGE;
   cudaStream_t s = (cudaStream_t)stream;
   (void)mode;
+#define AYK_GA(T, S)                                                                           \
+  return gated_attention<T, S>(q, ld_q, k_pages, v_pages, block_table, ld_table,               \
+                               request_of_row, positions, gate, ld_gate, out, ld_out, rows,    \
+                               heads, kv_heads, dim, vdim, page_size, scale, window,           \
+                               keep_first, slope, score_bias, s)
   if (type == 0) {
-    return gated_attention<float>(q, ld_q, k_pages, v_pages, block_table, ld_table,
-                                  request_of_row, positions, gate, ld_gate, out, ld_out, rows,
-                                  heads, kv_heads, dim, vdim, page_size, scale, window,
-                                  keep_first, s);
+    if (scores == SCORES_SIGMOID) AYK_GA(float, SCORES_SIGMOID);
+    if (scores == SCORES_SLOPED) AYK_GA(float, SCORES_SLOPED);
+    AYK_GA(float, SCORES_SOFTMAX);
   }
-  if (type == 1) {
-    return gated_attention<__nv_bfloat16>(q, ld_q, k_pages, v_pages, block_table, ld_table,
-                                          request_of_row, positions, gate, ld_gate, out, ld_out,
-                                          rows, heads, kv_heads, dim, vdim, page_size, scale,
-                                          window, keep_first, s);
-  }
-  return AYK_BAD_ARGUMENT;
+  if (scores == SCORES_SIGMOID) AYK_GA(__nv_bfloat16, SCORES_SIGMOID);
+  if (scores == SCORES_SLOPED) AYK_GA(__nv_bfloat16, SCORES_SLOPED);
+  AYK_GA(__nv_bfloat16, SCORES_SOFTMAX);
+#undef AYK_GA
 }

@@ -25,21 +25,22 @@ namespace ayk {
 //   latent page row <- [ c_raw * rsqrt(mean(c_raw^2) + eps) * w_c | rotate(kr_raw) ]
 //   q_plain[row]    <- the heads' unrotated parts            [heads x dim]
 //   qa[row]         <- rotate(q_rot) at [h][rank ..]          [heads x (rank + rot)]
-// Only the first rot_dims entries of a rotated piece are turned; the rest passes.
+// Only the first rot_dims entries of a rotated piece are turned; the rest passes. Cosines and
+// sines are multiplied by rot_gain.
 template <typename T>
 __global__ void latent_prepare_kernel(const float* __restrict__ proj, int ld_proj, int kv_offset,
                                       const float* __restrict__ latent_weight, float eps,
                                       const int* __restrict__ positions,
                                       const int* __restrict__ slots,
-                                      const double* __restrict__ freq, int rot_dims, int layout,
-                                      T* __restrict__ pages, T* __restrict__ q_plain,
-                                      int ld_plain, T* __restrict__ qa, int ld_qa, int heads,
-                                      int dim, int rot, int rank) {
+                                      const double* __restrict__ freq, int rot_dims,
+                                      float rot_gain, int layout, T* __restrict__ pages,
+                                      T* __restrict__ q_plain, int ld_plain, T* __restrict__ qa,
+                                      int ld_qa, int heads, int dim, int rot, int rank) {
   __shared__ float cos_s[ROPE_MAX_PAIRS], sin_s[ROPE_MAX_PAIRS];
   __shared__ float scratch[33];
   pdl_launch_dependents();
   const int row = blockIdx.x, pairs = rot_dims / 2;
-  rope_fill_table(cos_s, sin_s, positions[row], freq, pairs);
+  rope_fill_table(cos_s, sin_s, positions[row], freq, pairs, rot_gain);
   const int slot = slots != nullptr ? slots[row] : -1;
   pdl_wait_for(proj);
   const float* src = proj + (size_t)row * ld_proj;
@@ -94,9 +95,10 @@ __global__ void latent_prepare_kernel(const float* __restrict__ proj, int ld_pro
 // One small product per head: out[n][h][j] = sum_i a[n][h][i] * W_h(i, j), fp32 sums in the
 // order of i whatever the batch. W_h(i, j) sits at w + h * w_head + i * w_in + j * w_out, so a
 // head's matrix is used as stored ([in, out] rows: w_in = cols, w_out = 1) or transposed
-// ([out, in] rows: w_in = 1, w_out = cols). With `gate` (fp32 [n][h * J + j]) the result is
-// multiplied by sigmoid(gate). Tiles go through shared memory a slice of the inner dimension
-// at a time.
+// ([out, in] rows: w_in = 1, w_out = cols). With `gate` (fp32: one per entry, [n][h * J + j], or
+// one per head, [n][h]; gate_head = J or 1 of them a head, gate_step = 1 or 0 apart from column to
+// column) the result is multiplied by sigmoid(gate). Tiles go through shared memory a slice of the
+// inner dimension at a time.
 constexpr int HL_BN = 64;
 
 // A CTA of 256 threads computes (256 / (BN / TN)) * TM rows x BN columns, BK of the inner
@@ -109,8 +111,8 @@ template <typename T, int TM, int TN, int BK, int BN = HL_BN>
 __global__ void __launch_bounds__(256)
 head_linear_kernel(const T* __restrict__ a, int ld_a, int a_head, const T* __restrict__ w,
                    long long w_head, int w_in, int w_out, const float* __restrict__ gate,
-                   int ld_gate, T* __restrict__ out, int ld_out, int out_head, int rows, int I,
-                   int J) {
+                   int ld_gate, int gate_head, int gate_step, T* __restrict__ out, int ld_out,
+                   int out_head, int rows, int I, int J) {
   constexpr int TX = BN / TN, TY = 256 / TX, BM = TY * TM;
   __shared__ float a_s[BK][BM + 1];
   __shared__ float w_s[BK][BN + 1];
@@ -165,7 +167,7 @@ head_linear_kernel(const T* __restrict__ a, int ld_a, int a_head, const T* __res
       if (n >= J) continue;
       float v = acc[r][c];
       if (gate != nullptr) {
-        const float z = gate[(size_t)m * ld_gate + (size_t)h * J + n];
+        const float z = gate[(size_t)m * ld_gate + (size_t)h * gate_head + n * gate_step];
         v *= 1.f / (1.f + expf(-z));
       }
       stf(out + (size_t)m * ld_out + (size_t)h * out_head + n, v);
@@ -218,9 +220,9 @@ template <bool K_ROWS>
 __global__ void __launch_bounds__(128)
 head_linear_mma_kernel(const __nv_bfloat16* __restrict__ a, int ld_a, int a_head,
                        const __nv_bfloat16* __restrict__ w, long long w_head, int ld_w,
-                       const float* __restrict__ gate, int ld_gate,
-                       __nv_bfloat16* __restrict__ out, int ld_out, int out_head, int rows,
-                       int I, int J) {
+                       const float* __restrict__ gate, int ld_gate, int gate_head,
+                       int gate_step, __nv_bfloat16* __restrict__ out, int ld_out, int out_head,
+                       int rows, int I, int J) {
   __shared__ __align__(16) __nv_bfloat16 a_s[2][HM_TILE * HM_STRIDE];
   __shared__ __align__(16) __nv_bfloat16 w_s[2][HM_TILE * HM_STRIDE];
   pdl_launch_dependents();
@@ -300,9 +302,9 @@ head_linear_mma_kernel(const __nv_bfloat16* __restrict__ a, int ld_a, int a_head
       if (m >= rows) continue;
       float v0 = acc[t][2 * half], v1 = acc[t][2 * half + 1];
       if (gate != nullptr) {
-        const float* z = gate + (size_t)m * ld_gate + (size_t)h * J + n;
+        const float* z = gate + (size_t)m * ld_gate + (size_t)h * gate_head + n * gate_step;
         v0 *= 1.f / (1.f + expf(-z[0]));
-        v1 *= 1.f / (1.f + expf(-z[1]));
+        v1 *= 1.f / (1.f + expf(-z[gate_step]));
       }
       *reinterpret_cast<uint32_t*>(out + (size_t)m * ld_out + (size_t)h * out_head + n) =
           lm_pack(v0, v1);
@@ -320,8 +322,8 @@ inline bool head_linear_mma_takes(const void* a, int ld_a, int a_head, const voi
 
 template <typename T>
 int head_linear(const void* a, int ld_a, int a_head, const void* w, long long w_head, int w_in,
-                int w_out, const float* gate, int ld_gate, void* out, int ld_out, int out_head,
-                int rows, int heads, int I, int J, cudaStream_t s) {
+                int w_out, const float* gate, int ld_gate, int gate_head, int gate_step, void* out,
+                int ld_out, int out_head, int rows, int heads, int I, int J, cudaStream_t s) {
   const int tiles = (J + HL_BN - 1) / HL_BN;
   if (tiles > 65535) return AYK_TOO_LARGE;
   if constexpr (std::is_same<T, __nv_bfloat16>::value) {
@@ -332,26 +334,29 @@ int head_linear(const void* a, int ld_a, int a_head, const void* w, long long w_
       if (w_in == 1) {
         return launch_kernel(head_linear_mma_kernel<true>, grid, dim3(128), 0, s, 1,
                              (const T*)a, ld_a, a_head, (const T*)w, w_head, ld_w, gate,
-                             ld_gate, (T*)out, ld_out, out_head, rows, I, J);
+                           ld_gate, gate_head, gate_step, (T*)out, ld_out, out_head, rows, I, J);
       }
       return launch_kernel(head_linear_mma_kernel<false>, grid, dim3(128), 0, s, 1,
-                           (const T*)a, ld_a, a_head, (const T*)w, w_head, ld_w, gate, ld_gate,
-                           (T*)out, ld_out, out_head, rows, I, J);
+                           (const T*)a, ld_a, a_head, (const T*)w, w_head, ld_w, gate,
+                           ld_gate, gate_head, gate_step, (T*)out, ld_out, out_head, rows, I, J);
     }
   }
   if (rows <= 16) {
     if (I > 64) {  // up to 256 of the inner dimension in one trip to memory
       return launch_kernel(head_linear_kernel<T, 1, 1, 256, 16>, dim3(1, (J + 15) / 16, heads),
                            dim3(256), 0, s, 1, (const T*)a, ld_a, a_head, (const T*)w, w_head,
-                           w_in, w_out, gate, ld_gate, (T*)out, ld_out, out_head, rows, I, J);
+                           w_in, w_out, gate, ld_gate, gate_head, gate_step, (T*)out, ld_out,
+                           out_head, rows, I, J);
     }
     return launch_kernel(head_linear_kernel<T, 1, 1, 64, 16>, dim3(1, (J + 15) / 16, heads),
                          dim3(256), 0, s, 1, (const T*)a, ld_a, a_head, (const T*)w, w_head,
-                         w_in, w_out, gate, ld_gate, (T*)out, ld_out, out_head, rows, I, J);
+                         w_in, w_out, gate, ld_gate, gate_head, gate_step, (T*)out, ld_out,
+                           out_head, rows, I, J);
   }
   return launch_kernel(head_linear_kernel<T, 2, 4, 16>, dim3((rows + 31) / 32, tiles, heads),
                        dim3(256), 0, s, 1, (const T*)a, ld_a, a_head, (const T*)w, w_head, w_in,
-                       w_out, gate, ld_gate, (T*)out, ld_out, out_head, rows, I, J);
+                       w_out, gate, ld_gate, gate_head, gate_step, (T*)out, ld_out,
+                           out_head, rows, I, J);
 }
 
 // ---------------------------------------------------------------------------------------------
@@ -362,6 +367,8 @@ int head_linear(const void* a, int ld_a, int a_head, const void* w, long long w_
 // over all rank + rot entries, the warp keeps a running maximum and sum (fp32, expf), then the
 // lanes split the first `rank` entries of the key rows and add w_j * row_j. The tiling depends
 // only on the position: a row's result is the same alone, in a portion or in a mixed batch.
+// With `sink` (one float per head) the softmax's denominator also holds exp(sink[head]): an entry
+// without key or value. A head's result starts every out_head columns.
 constexpr int LA_WARPS = 4;
 
 template <typename T> struct Chunk8;
@@ -391,8 +398,9 @@ latent_attention_kernel(const T* __restrict__ qa, int ld_qa, const T* __restrict
                         const int* __restrict__ block_table, int table_stride,
                         const int* __restrict__ request_of_row,
                         const int* __restrict__ positions, T* __restrict__ out, int ld_out,
-                        int num_heads, int rank, int key_dim, int key_pad, int page_size,
-                        float scale, int window, int vector_ok) {
+                        int out_head, int num_heads, int rank, int key_dim, int key_pad,
+                        int page_size, float scale, int window, const float* __restrict__ sink,
+                        int vector_ok) {
   extern __shared__ __align__(16) float la_smem[];
   float* q_s = la_smem + (size_t)(threadIdx.x >> 5) * key_pad;
   __shared__ float w_s[LA_WARPS][32];
@@ -403,7 +411,7 @@ latent_attention_kernel(const T* __restrict__ qa, int ld_qa, const T* __restrict
   if (head >= num_heads) return;  // (no block barrier below)
   const int b = request_of_row[row], p = positions[row];
   pdl_wait_for(qa, pages);
-  T* dst = out + (size_t)row * ld_out + (size_t)head * rank;
+  T* dst = out + (size_t)row * ld_out + (size_t)head * out_head;
   if (b < 0) {
     for (int d = lane; d < rank; d += 32) stf(dst + d, 0.f);
     return;
@@ -462,7 +470,11 @@ latent_attention_kernel(const T* __restrict__ qa, int ld_qa, const T* __restrict
     }
     __syncwarp();
   }
-  const float inv = 1.f / l;
+  float inv = 1.f / l;
+  if (sink != nullptr) {
+    const float top = fmaxf(m, sink[head]), corr = expf(m - top);
+    inv = corr / (l * corr + expf(sink[head] - top));
+  }
 #pragma unroll
   for (int r = 0; r < R; ++r) {
     const int d = lane + 32 * r;
@@ -619,7 +631,8 @@ constexpr int LD_MAX_SPLITS = 64;
 template <typename T>
 __global__ void latent_decode_merge_kernel(const float* __restrict__ partial,
                                            T* __restrict__ out, int ld_out, int out_head,
-                                           int num_heads, int rank, int splits) {
+                                           int num_heads, int rank, int splits,
+                                           const float* __restrict__ sink) {
   __shared__ float max_s[LD_MAX_SPLITS], weight_s[LD_MAX_SPLITS];
   pdl_launch_dependents();
   const int row = blockIdx.x, head = blockIdx.y;
@@ -636,6 +649,13 @@ __global__ void latent_decode_merge_kernel(const float* __restrict__ partial,
   for (int s = 0; s < splits; ++s) {  // (a share without keys has sum 0 and maximum -inf)
     l += weight_s[s] > 0.f ? weight_s[s] * expf(max_s[s] - m) : 0.f;
   }
+  // the sink: one more entry of the denominator, counted once, where the shares meet
+  float scaled = 1.f;
+  if (sink != nullptr && l > 0.f) {
+    const float top = fmaxf(m, sink[head]);
+    scaled = expf(m - top);
+    l = l * scaled + expf(sink[head] - top);
+  }
   __syncthreads();
   for (int s = threadIdx.x; s < splits; s += blockDim.x) {
     weight_s[s] = weight_s[s] > 0.f ? expf(max_s[s] - m) : 0.f;
@@ -646,7 +666,7 @@ __global__ void latent_decode_merge_kernel(const float* __restrict__ partial,
     float v = 0.f;
 #pragma unroll 8
     for (int s = 0; s < splits; ++s) v = fmaf(from[(size_t)s * (rank + 2) + 2 + d], weight_s[s], v);
-    stf(dst + d, l > 0.f ? v / l : 0.f);
+    stf(dst + d, l > 0.f ? v * scaled / l : 0.f);
   }
 }
 
@@ -864,8 +884,9 @@ latent_decode_mma_kernel(const __nv_bfloat16* __restrict__ qa, int ld_qa,
 template <typename T>
 int latent_attention(const void* qa, int ld_qa, const void* pages, const int* block_table,
                      int table_stride, const int* request_of_row, const int* positions, void* out,
-                     int ld_out, int rows, int num_heads, int rank, int rot, int page_size,
-                     float scale, int window, cudaStream_t stream) {
+                     int ld_out, int out_head, int rows, int num_heads, int rank, int rot,
+                     int page_size, float scale, int window, const float* sink,
+                     cudaStream_t stream) {
   const int key_dim = rank + rot;
   const int key_pad = (key_dim + 7) / 8 * 8;
   const int vector_ok =
@@ -875,8 +896,8 @@ int latent_attention(const void* qa, int ld_qa, const void* pages, const int* bl
 #define AYK_LA(R)                                                                              \
   return launch_kernel(latent_attention_kernel<T, R>, grid, block, smem, stream, 1,            \
                        (const T*)qa, ld_qa, (const T*)pages, block_table, table_stride,        \
-                       request_of_row, positions, (T*)out, ld_out, num_heads, rank, key_dim,   \
-                       key_pad, page_size, scale, window, vector_ok)
+                       request_of_row, positions, (T*)out, ld_out, out_head, num_heads, rank,  \
+                       key_dim, key_pad, page_size, scale, window, sink, vector_ok)
   if (rank <= 64) AYK_LA(2);
   if (rank <= 128) AYK_LA(4);
   if (rank <= 256) AYK_LA(8);
@@ -897,10 +918,10 @@ AYK_API void ayk_set_latent_decode_tensor_cores(int on) { ayk::decode_tensor_cor
 // cache another run wrote) or a row's slot negative: nothing is stored then.
 AYK_API int ayk_latent_prepare(const float* proj, int ld_proj, int kv_offset,
                                const float* latent_weight, float eps, const int* positions,
-                               const int* slots, const double* freq, int rot_dims, int layout,
-                               void* pages, void* q_plain, int ld_plain, void* qa, int ld_qa,
-                               int rows, int heads, int dim, int rot, int rank, int type,
-                               void* stream) {
+                               const int* slots, const double* freq, int rot_dims, float rot_gain,
+                               int layout, void* pages, void* q_plain, int ld_plain, void* qa,
+                               int ld_qa, int rows, int heads, int dim, int rot, int rank,
+                               int type, void* stream) {
   using namespace ayk;
   if (rows == 0) return AYK_OK;
   if (rows < 0 || heads < 1 || dim < 0 || rot < 0 || rank < 1 || rot_dims < 0 || rot_dims % 2 ||
@@ -917,36 +938,42 @@ AYK_API int ayk_latent_prepare(const float* proj, int ld_proj, int kv_offset,
   if (type == 0) {
     return launch_kernel(latent_prepare_kernel<float>, dim3(rows), dim3(256), 0, s, 1, proj,
                          ld_proj, kv_offset, latent_weight, eps, positions, slots, freq, rot_dims,
-                         layout, (float*)pages, (float*)q_plain, ld_plain, (float*)qa, ld_qa,
-                         heads, dim, rot, rank);
+                         rot_gain, layout, (float*)pages, (float*)q_plain, ld_plain, (float*)qa,
+                         ld_qa, heads, dim, rot, rank);
   }
   if (type == 1) {
     return launch_kernel(latent_prepare_kernel<__nv_bfloat16>, dim3(rows), dim3(256), 0, s, 1,
-                         proj, ld_proj, kv_offset, latent_weight, eps, positions, slots, freq,
-                         rot_dims, layout, (__nv_bfloat16*)pages, (__nv_bfloat16*)q_plain,
-                         ld_plain, (__nv_bfloat16*)qa, ld_qa, heads, dim, rot, rank);
+                         proj, ld_proj, kv_offset, latent_weight, eps, positions, slots,
+                         freq, rot_dims, rot_gain, layout, (__nv_bfloat16*)pages,
+                         (__nv_bfloat16*)q_plain, ld_plain, (__nv_bfloat16*)qa, ld_qa, heads, dim,
+                         rot, rank);
   }
   return AYK_BAD_ARGUMENT;
 }
 
+// `gate` (may be null) has gate_head entries per head, 1 (one gate for all of a head's columns) or
+// J.
 AYK_API int ayk_head_linear(const void* a, int ld_a, int a_head, const void* w, long long w_head,
-                            int w_in, int w_out, const float* gate, int ld_gate, void* out,
-                            int ld_out, int out_head, int rows, int heads, int I, int J, int type,
-                            void* stream) {
+                            int w_in, int w_out, const float* gate, int ld_gate, int gate_head,
+                            void* out, int ld_out, int out_head, int rows, int heads, int I,
+                            int J, int type, void* stream) {
   using namespace ayk;
   if (rows == 0 || heads == 0 || J == 0) return AYK_OK;
   if (rows < 0 || heads < 0 || I < 1 || J < 0 || a == nullptr || w == nullptr || out == nullptr ||
-      w_in < 1 || w_out < 1 || (w_in != 1 && w_out != 1) || heads > 65535) {
+      w_in < 1 || w_out < 1 || (w_in != 1 && w_out != 1) || heads > 65535 ||
+      (gate != nullptr && ((gate_head != 1 && gate_head != J) || ld_gate < heads * gate_head))) {
     return AYK_BAD_ARGUMENT;
   }
+  const int gate_step = gate_head == J ? 1 : 0;
   cudaStream_t s = (cudaStream_t)stream;
   if (type == 0) {
-    return head_linear<float>(a, ld_a, a_head, w, w_head, w_in, w_out, gate, ld_gate, out, ld_out,
-                              out_head, rows, heads, I, J, s);
+    return head_linear<float>(a, ld_a, a_head, w, w_head, w_in, w_out, gate, ld_gate, gate_head,
+                              gate_step, out, ld_out, out_head, rows, heads, I, J, s);
   }
   if (type == 1) {
-    return head_linear<__nv_bfloat16>(a, ld_a, a_head, w, w_head, w_in, w_out, gate, ld_gate, out,
-                                      ld_out, out_head, rows, heads, I, J, s);
+    return head_linear<__nv_bfloat16>(a, ld_a, a_head, w, w_head, w_in, w_out, gate, ld_gate,
+                                      gate_head, gate_step, out, ld_out, out_head, rows, heads, I,
+                                      J, s);
   }
   return AYK_BAD_ARGUMENT;
 }
@@ -954,27 +981,28 @@ AYK_API int ayk_head_linear(const void* a, int ld_a, int a_head, const void* w, 
 AYK_API int ayk_latent_attention(const void* qa, int ld_qa, const void* pages,
                                  const int* block_table, int table_stride,
                                  const int* request_of_row, const int* positions, void* out,
-                                 int ld_out, int rows, int num_heads, int rank, int rot,
-                                 int page_size, float scale, int window, int type, void* stream) {
+                                 int ld_out, int out_head, int rows, int num_heads, int rank,
+                                 int rot, int page_size, float scale, int window,
+                                 const float* sink, int type, void* stream) {
   using namespace ayk;
   if (rows == 0) return AYK_OK;
   if (rows < 0 || num_heads < 1 || rank < 1 || rot < 0 || page_size < 1 || window < 0 ||
       qa == nullptr || pages == nullptr || block_table == nullptr || request_of_row == nullptr ||
       positions == nullptr || out == nullptr || ld_qa < num_heads * (rank + rot) ||
-      ld_out < num_heads * rank) {
+      out_head < rank || ld_out < (num_heads - 1) * out_head + rank) {
     return AYK_BAD_ARGUMENT;
   }
   if (rank > 1024 || rank + rot > 2048 || num_heads > 65535 * ayk::LA_WARPS) return AYK_TOO_LARGE;
   cudaStream_t s = (cudaStream_t)stream;
   if (type == 0) {
     return latent_attention<float>(qa, ld_qa, pages, block_table, table_stride, request_of_row,
-                                   positions, out, ld_out, rows, num_heads, rank, rot, page_size,
-                                   scale, window, s);
+                                   positions, out, ld_out, out_head,
+                                   rows, num_heads, rank, rot, page_size, scale, window, sink, s);
   }
   if (type == 1) {
     return latent_attention<__nv_bfloat16>(qa, ld_qa, pages, block_table, table_stride,
-                                           request_of_row, positions, out, ld_out, rows, num_heads,
-                                           rank, rot, page_size, scale, window, s);
+                                           request_of_row, positions, out, ld_out, out_head,
+                                   rows, num_heads, rank, rot, page_size, scale, window, sink, s);
   }
   return AYK_BAD_ARGUMENT;
 }
@@ -989,7 +1017,7 @@ AYK_API int ayk_latent_decode(const void* qa, int ld_qa, const void* pages,
                               const int* request_of_row, const int* positions, float* partial,
                               void* out, int ld_out, int out_head, int rows, int num_heads,
                               int rank, int rot, int page_size, float scale, int window,
-                              int splits, int type, void* stream) {
+                              const float* sink, int splits, int type, void* stream) {
   using namespace ayk;
   if (rows == 0) return AYK_OK;
   const int key_dim = rank + rot;
@@ -1030,7 +1058,7 @@ AYK_API int ayk_latent_decode(const void* qa, int ld_qa, const void* pages,
     if (status != AYK_OK) return status;
     return launch_kernel(latent_decode_merge_kernel<__nv_bfloat16>, dim3(rows, num_heads),
                          dim3(128), 0, s, 1, (const float*)partial, (__nv_bfloat16*)out, ld_out,
-                         out_head, num_heads, rank, splits);
+                         out_head, num_heads, rank, splits, sink);
   }
   const int elem = type == 0 ? 4 : 2;
   const int group = LD_WARPS * LD_HEADS;
@@ -1049,7 +1077,7 @@ AYK_API int ayk_latent_decode(const void* qa, int ld_qa, const void* pages,
     if (status != AYK_OK) return status;
     return launch_kernel(latent_decode_merge_kernel<float>, dim3(rows, num_heads), dim3(128), 0,
                          s, 1, (const float*)partial, (float*)out, ld_out, out_head, num_heads,
-                         rank, splits);
+                         rank, splits, sink);
   }
   static const bool allowed = (cudaFuncSetAttribute(
       latent_decode_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize,
@@ -1062,5 +1090,5 @@ AYK_API int ayk_latent_decode(const void* qa, int ld_qa, const void* pages,
   if (status != AYK_OK) return status;
   return launch_kernel(latent_decode_merge_kernel<__nv_bfloat16>, dim3(rows, num_heads),
                        dim3(128), 0, s, 1, (const float*)partial, (__nv_bfloat16*)out, ld_out,
-                       out_head, num_heads, rank, splits);
+                       out_head, num_heads, rank, splits, sink);
 }

@@ -332,8 +332,12 @@ __global__ void norm_sum_kernel(Branches in, int count, float eps, float factor,
 // When `next_out` is given, also next_out[r][c] = v[c] * rsqrt(mean_c(v^2) + next_eps) *
 // (next_offset + next_weight[c]) with v the new dst[r]: the norm in front of the next sublayer,
 // from the row that is in registers anyway (one more sum over the row, no launch of its own).
+// When `other` is given, x stands for x_factor * x + other_factor * other (two mixers side by side
+// whose weighted sum is normed as one result).
 template <typename TOut>
-__global__ void norm_add_kernel(const float* __restrict__ x, int ld_x,
+__global__ void norm_add_kernel(const float* __restrict__ x, int ld_x, float x_factor,
+                                const float* __restrict__ other, int ld_other,
+                                float other_factor,
                                 const float* __restrict__ weight, float offset, float eps,
                                 float factor, float* __restrict__ dst, int ld_dst,
                                 TOut* __restrict__ copy, int ld_copy, int width,
@@ -353,7 +357,7 @@ __global__ void norm_add_kernel(const float* __restrict__ x, int ld_x,
       const int c = threadIdx.x + i * blockDim.x;
       ws[i] = c < width ? offset + weight[c] : 0.f;
     }
-    pdl_wait_for(x, dst);
+    pdl_wait_for(x, dst, other);
     const float* src = x + (size_t)r * ld_x;
     float* to = dst + (size_t)r * ld_dst;
     float s = 0.f;
@@ -362,6 +366,14 @@ __global__ void norm_add_kernel(const float* __restrict__ x, int ld_x,
       const int c = threadIdx.x + i * blockDim.x;
       xs[i] = c < width ? src[c] : 0.f;
       ds[i] = c < width ? to[c] : 0.f;
+    }
+    if (other != nullptr) {
+      const float* src2 = other + (size_t)r * ld_other;
+#pragma unroll
+      for (int i = 0; i < NA_KEEP; ++i) {
+        const int c = threadIdx.x + i * blockDim.x;
+        xs[i] = xs[i] * x_factor + (c < width ? src2[c] : 0.f) * other_factor;
+      }
     }
 #pragma unroll
     for (int i = 0; i < NA_KEEP; ++i) s += xs[i] * xs[i];
@@ -390,15 +402,19 @@ __global__ void norm_add_kernel(const float* __restrict__ x, int ld_x,
     }
     return;
   }
-  pdl_wait_for(x, dst);
+  pdl_wait_for(x, dst, other);
   const float* src = x + (size_t)r * ld_x;
+  auto entry = [&](int c) {
+    return other == nullptr ? src[c]
+                            : src[c] * x_factor + other[(size_t)r * ld_other + c] * other_factor;
+  };
   float s = 0.f;
-  for (int c = threadIdx.x; c < width; c += blockDim.x) s += src[c] * src[c];
+  for (int c = threadIdx.x; c < width; c += blockDim.x) s += entry(c) * entry(c);
   const float inv = factor / sqrtf(block_sum(s, scratch) / (float)width + eps);
   float* to = dst + (size_t)r * ld_dst;
   float s2 = 0.f;
   for (int c = threadIdx.x; c < width; c += blockDim.x) {
-    const float v = to[c] + src[c] * inv * (offset + weight[c]);
+    const float v = to[c] + entry(c) * inv * (offset + weight[c]);
     to[c] = v;
     if (copy != nullptr) stf(copy + (size_t)r * ld_copy + c, v);
     s2 += v * v;
@@ -483,7 +499,9 @@ AYK_API int ayk_scale_add(const float* x, int ld_x, const float* scale, float* d
 
 // copy_type: 0 = float32, 1 = bfloat16, of `copy` and of `next_out` (ignored when both are
 // null). `next_out` with `next_weight`: the following norm's output (see norm_add_kernel).
-AYK_API int ayk_norm_add_next(const float* x, int ld_x, const float* weight, float offset,
+// `other` (may be null) joins x first: x_factor * x + other_factor * other.
+AYK_API int ayk_norm_add_next(const float* x, int ld_x, float x_factor, const float* other,
+                              int ld_other, float other_factor, const float* weight, float offset,
                               float eps, float factor, float* dst, int ld_dst, void* copy,
                               int ld_copy, int copy_type, const float* next_weight,
                               float next_offset, float next_eps, void* next_out, int ld_next,
@@ -492,6 +510,7 @@ AYK_API int ayk_norm_add_next(const float* x, int ld_x, const float* weight, flo
   if (n == 0) return AYK_OK;
   if (n < 0 || width < 1 || x == nullptr || weight == nullptr || dst == nullptr ||
       ld_x < width || ld_dst < width || (copy != nullptr && ld_copy < width) || !(eps > 0.f) ||
+      (other != nullptr && ld_other < width) ||
       (next_out != nullptr && (next_weight == nullptr || ld_next < width ||
                                !(next_eps > 0.f)))) {
     return AYK_BAD_ARGUMENT;
@@ -500,20 +519,22 @@ AYK_API int ayk_norm_add_next(const float* x, int ld_x, const float* weight, flo
   const bool typed = copy != nullptr || next_out != nullptr;
   if (typed && copy_type == 1) {
     return launch_kernel(norm_add_kernel<__nv_bfloat16>, dim3(n), dim3(threads), 0,
-                         (cudaStream_t)stream, 1, x, ld_x, weight, offset, eps, factor, dst,
-                         ld_dst, (__nv_bfloat16*)copy, ld_copy, width, next_weight, next_offset,
-                         next_eps, (__nv_bfloat16*)next_out, ld_next);
+                         (cudaStream_t)stream, 1, x, ld_x, x_factor, other, ld_other,
+                         other_factor, weight, offset, eps, factor, dst, ld_dst,
+                         (__nv_bfloat16*)copy, ld_copy, width, next_weight, next_offset, next_eps,
+                         (__nv_bfloat16*)next_out, ld_next);
   }
   if (typed && copy_type != 0) return AYK_BAD_ARGUMENT;
   return launch_kernel(norm_add_kernel<float>, dim3(n), dim3(threads), 0, (cudaStream_t)stream,
-                       1, x, ld_x, weight, offset, eps, factor, dst, ld_dst, (float*)copy,
-                       ld_copy, width, next_weight, next_offset, next_eps, (float*)next_out,
-                       ld_next);
+                       1, x, ld_x, x_factor, other, ld_other, other_factor, weight, offset, eps,
+                       factor, dst, ld_dst, (float*)copy, ld_copy, width, next_weight,
+                       next_offset, next_eps, (float*)next_out, ld_next);
 }
 
 AYK_API int ayk_norm_add(const float* x, int ld_x, const float* weight, float offset, float eps,
                          float factor, float* dst, int ld_dst, void* copy, int ld_copy,
                          int copy_type, int n, int width, void* stream) {
-  return ayk_norm_add_next(x, ld_x, weight, offset, eps, factor, dst, ld_dst, copy, ld_copy,
-                           copy_type, nullptr, 0.f, 1.f, nullptr, 0, n, width, stream);
+  return ayk_norm_add_next(x, ld_x, 1.f, nullptr, 0, 0.f, weight, offset, eps, factor, dst, ld_dst,
+                           copy, ld_copy, copy_type, nullptr, 0.f, 1.f, nullptr, 0, n, width,
+                           stream);
 }

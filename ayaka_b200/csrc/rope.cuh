@@ -15,14 +15,16 @@ namespace ayk {
 constexpr int ROPE_MAX_PAIRS = 256;
 enum RopeLayout : int { ROPE_NEIGHBOURS = 0, ROPE_HALVES = 1 };
 
-// cos_s, sin_s: ROPE_MAX_PAIRS floats each in shared memory; a barrier must follow.
+// cos_s, sin_s: ROPE_MAX_PAIRS floats each in shared memory; a barrier must follow. Both are
+// multiplied by `gain`.
 __device__ __forceinline__ void rope_fill_table(float* cos_s, float* sin_s, int position,
-                                                const double* __restrict__ freq, int pairs) {
+                                                const double* __restrict__ freq, int pairs,
+                                                float gain = 1.f) {
   for (int i = threadIdx.x; i < pairs; i += blockDim.x) {
     double s, c;
     sincos((double)position * freq[i], &s, &c);
-    cos_s[i] = (float)c;
-    sin_s[i] = (float)s;
+    cos_s[i] = (float)c * gain;
+    sin_s[i] = (float)s * gain;
   }
 }
 

@@ -476,7 +476,9 @@ def attention_prefill(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Ten
                       window: int = 0, kernel: str | None = None, keep_first: int = 0,
                       gate: torch.Tensor | None = None, pool: int = 0,
                       k_pool: torch.Tensor | None = None, v_pool: torch.Tensor | None = None,
-                      sink: torch.Tensor | None = None) -> None:
+                      sink: torch.Tensor | None = None, scores: str = "softmax",
+                      slope: torch.Tensor | None = None,
+                      score_bias: torch.Tensor | None = None) -> None:
     """Causal attention of prompt portions in bfloat16 on the tensor cores.
 
     Request ``b`` owns rows ``row_start[b] .. row_start[b + 1]`` of ``q`` and ``out``, which
@@ -489,6 +491,8 @@ def attention_prefill(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Ten
     with ``pool`` and a window the pooled rows ``k_pool`` / ``v_pool`` of the blocks that lie
     wholly behind a row's window (see :func:`pooled_attention`), and with ``sink`` (float32
     ``[num_heads]``) one more entry ``exp(sink[head])`` in the softmax's denominator.
+    ``scores``, ``slope`` and ``score_bias`` as in :func:`gated_attention` (a library compiled for
+    them; without pooled rows, a sigmoid without a sink).
     """
     op = "attention_prefill"
     if _left_out and op in _left_out:
@@ -529,16 +533,19 @@ def attention_prefill(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Ten
         _need(op, "sink", sink, torch.float32, 1)
         if sink.shape[0] != num_heads:
             raise BackendError(f"{op}: one sink per head")
+    mode = _need_scores(op, scores, slope, score_bias, num_heads)
+    if (mode and pooled) or (scores == "sigmoid" and sink is not None):
+        raise BackendError(f"{op}: slopes do not go with pooled rows, a sigmoid not with a sink")
     plain = value_dim == head_dim and gate is None and not (keep_first and window) and \
-        not pooled and sink is None
+        not pooled and sink is None and not mode
     # the tcgen05 kernel works on tiles of 256 rows: a step of short portions only is better
     # served by the warp-level kernel's tiles of 64
     which = kernel or (PREFILL_ATTENTION if head_dim == 64 and scale > 0 and plain
                        and max(host_rows, default=0) >= 256 else "mma")
     if which == "tcgen05":
         if head_dim != 64 or not plain:
-            raise BackendError(f"{op}: the tcgen05 kernel serves head size 64 without a gate, "
-                               f"kept keys or value rows of their own, not {head_dim}")
+            raise BackendError(f"{op}: the tcgen05 kernel serves a softmax of head size 64 without "
+                               f"a gate, kept keys, value rows of their own, not {head_dim}")
         lib = library("attention_prefill_tc")
         tile_rows = lib.ayk_attention_prefill_tc_rows()
         tiles = sum(-(-rows // tile_rows) for rows in host_rows)
@@ -554,6 +561,8 @@ def attention_prefill(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Ten
     sizes = {"AYK_HEAD_DIM": head_dim}
     if value_dim != head_dim:
         sizes["AYK_VALUE_DIM"] = value_dim
+    if mode:
+        sizes["AYK_SCORES"] = mode
     fn = library("attention_prefill", **sizes).ayk_attention_prefill_pooled
     status = fn(_ptr(q), c_int(q.stride(0)), _ptr(k_pages), _ptr(v_pages), _ptr(block_table),
                 c_int(block_table.stride(0)), _ptr(row_start), _ptr(kv_len), _ptr(out),
@@ -563,7 +572,7 @@ def attention_prefill(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Ten
                 c_int(0 if gate is None else gate.stride(0)),
                 c_int(pool if pooled else 0), c_int(pool_slots(page_size, pool) if pooled else 0),
                 _ptr(k_pool if pooled else None), _ptr(v_pool if pooled else None), _ptr(sink),
-                _stream())
+                _ptr(slope), _ptr(score_bias), _stream())
     check(status, op)
 
 
@@ -888,13 +897,14 @@ def latent_prepare(proj: torch.Tensor, *, kv_offset: int, latent_weight: torch.T
                    eps: float, positions: torch.Tensor, slot_mapping: torch.Tensor | None,
                    freq: torch.Tensor, layout: str, pages: torch.Tensor | None,
                    q_plain: torch.Tensor, qa: torch.Tensor, heads: int, dim: int, rot: int,
-                   rank: int, rows: int) -> None:
+                   rank: int, rows: int, rot_gain: float = 1.0) -> None:
     """From a row of the fused projection (float32: the heads' queries ``[dim | rot]``, then
     at ``kv_offset`` the raw latent of ``rank`` entries and the raw shared key piece of
     ``rot``): the latent normalised by its root mean square times ``latent_weight`` and the
     rotated key piece go to the row's cache slot (``pages`` ``[page, 1, slot, rank + rot]``),
     the unrotated query parts to ``q_plain`` ``[N, heads * dim]``, the rotated ones to
-    ``qa[:, h, rank:]`` (``qa`` is ``[N, heads * (rank + rot)]``). Without ``pages`` (a layer
+    ``qa[:, h, rank:]`` (``qa`` is ``[N, heads * (rank + rot)]``); cosines and sines are
+    multiplied by ``rot_gain``. Without ``pages`` (a layer
     that reads latents another layer stored) the columns from ``kv_offset`` on are not read."""
     op = "latent_prepare"
     if _left_out and op in _left_out:
@@ -924,7 +934,8 @@ def latent_prepare(proj: torch.Tensor, *, kv_offset: int, latent_weight: torch.T
     status = library("latent_attention").ayk_latent_prepare(
         _ptr(proj), c_int(proj.stride(0)), c_int(kv_offset), _ptr(latent_weight), c_float(eps),
         _ptr(positions), _ptr(slot_mapping if pages is not None else None), _ptr(freq),
-        c_int(2 * freq.shape[0]), c_int(ROPE_LAYOUTS[layout]), _ptr(pages), _ptr(q_plain),
+        c_int(2 * freq.shape[0]), c_float(rot_gain), c_int(ROPE_LAYOUTS[layout]), _ptr(pages),
+        _ptr(q_plain),
         c_int(q_plain.stride(0)), _ptr(qa), c_int(qa.stride(0)), c_int(rows), c_int(heads),
         c_int(dim), c_int(rot), c_int(rank), c_int(_TYPE[q_plain.dtype]), _stream())
     check(status, op)
@@ -940,7 +951,8 @@ def head_linear(a: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, *, hea
     results start every ``out.shape[1] / heads`` columns). ``weight`` holds the heads' matrices
     one under the other: ``[heads * J, I]`` applied as ``W_h a_h`` (``transposed=False``), or
     ``[heads * I, J]`` applied as ``W_h^T a_h`` (``transposed=True``). With ``gate`` (float32
-    ``[N, heads * J]``) the result is multiplied by ``sigmoid(gate)``."""
+    ``[N, heads * J]``, or ``[N, heads]``: one for all of a head's results) the result is
+    multiplied by ``sigmoid(gate)``."""
     op = "head_linear"
     if _left_out and op in _left_out:
         return
@@ -968,12 +980,13 @@ def head_linear(a: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, *, hea
         raise BackendError(f"{op}: shapes do not fit")
     if gate is not None:
         _need(op, "gate", gate, torch.float32, 2)
-        if gate.shape[1] != heads * outer or gate.shape[0] < rows:
+        if gate.shape[1] not in (heads, heads * outer) or gate.shape[0] < rows:
             raise BackendError(f"{op}: the gate does not match the result")
     status = library("latent_attention").ayk_head_linear(
         _ptr(a), c_int(a.stride(0)), c_int(a_head), _ptr(weight),
         c_longlong(weight.shape[0] // heads * weight.shape[1]), c_int(w_in), c_int(w_out),
-        _ptr(gate), c_int(0 if gate is None else gate.stride(0)), _ptr(out),
+        _ptr(gate), c_int(0 if gate is None else gate.stride(0)),
+        c_int(0 if gate is None else gate.shape[1] // heads), _ptr(out),
         c_int(out.stride(0)), c_int(out_head), c_int(rows), c_int(heads), c_int(inner),
         c_int(outer), c_int(_TYPE[a.dtype]), _stream())
     check(status, op)
@@ -982,12 +995,14 @@ def head_linear(a: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, *, hea
 def latent_attention(qa: torch.Tensor, pages: torch.Tensor, block_table: torch.Tensor,
                      request_of_row: torch.Tensor, positions: torch.Tensor, out: torch.Tensor,
                      *, num_heads: int, rank: int, scale: float, window: int = 0,
-                     rows: int | None = None) -> None:
+                     rows: int | None = None, sink: torch.Tensor | None = None) -> None:
     """Attention of all heads over one latent row per token: the row of request
     ``request_of_row[i]`` at ``positions[i]`` scores ``scale * qa[i, h] . page_row`` over keys
     ``max(0, p - window + 1) .. p`` (``window`` 0: all) and returns the softmax-weighted sum of
-    the page rows' first ``rank`` entries: ``out`` is ``[N, num_heads * rank]``. ``pages`` is
-    ``[page, 1, slot, rank + rot]``; the step's own rows must already be stored."""
+    the page rows' first ``rank`` entries into the first ``rank`` of the head's ``out.shape[1] /
+    num_heads`` columns. With ``sink`` (float32 ``[num_heads]``) the softmax's denominator also
+    holds ``exp(sink[head])``. ``pages`` is ``[page, 1, slot, rank + rot]``; the step's own rows
+    must already be stored."""
     op = "latent_attention"
     if _left_out and op in _left_out:
         return
@@ -1001,16 +1016,25 @@ def latent_attention(qa: torch.Tensor, pages: torch.Tensor, block_table: torch.T
         raise BackendError(f"{op}: contiguous float32 or bfloat16 pages [page, 1, slot, row]")
     _, _, page_size, key_dim = pages.shape
     n = qa.shape[0] if rows is None else rows
-    if qa.shape[1] != num_heads * key_dim or out.shape[1] != num_heads * rank or \
-            rank > key_dim or n > out.shape[0] or n > request_of_row.shape[0] or \
-            n > positions.shape[0]:
+    if qa.shape[1] != num_heads * key_dim or out.shape[1] % num_heads or \
+            out.shape[1] // num_heads < rank or rank > key_dim or n > out.shape[0] or \
+            n > request_of_row.shape[0] or n > positions.shape[0]:
         raise BackendError(f"{op}: shapes do not fit")
+    _need_sink(op, sink, num_heads)
     status = library("latent_attention").ayk_latent_attention(
         _ptr(qa), c_int(qa.stride(0)), _ptr(pages), _ptr(block_table),
         c_int(block_table.stride(0)), _ptr(request_of_row), _ptr(positions), _ptr(out),
-        c_int(out.stride(0)), c_int(n), c_int(num_heads), c_int(rank), c_int(key_dim - rank),
-        c_int(page_size), c_float(scale), c_int(window), c_int(_TYPE[qa.dtype]), _stream())
+        c_int(out.stride(0)), c_int(out.shape[1] // num_heads), c_int(n), c_int(num_heads),
+        c_int(rank), c_int(key_dim - rank), c_int(page_size), c_float(scale), c_int(window),
+        _ptr(sink), c_int(_TYPE[qa.dtype]), _stream())
     check(status, op)
+
+
+def _need_sink(op: str, sink: torch.Tensor | None, heads: int) -> None:
+    if sink is not None:
+        _need(op, "sink", sink, torch.float32, 1)
+        if sink.shape[0] != heads:
+            raise BackendError(f"{op}: one sink per head")
 
 
 def set_latent_decode_tensor_cores(enabled: bool) -> None:
@@ -1036,7 +1060,8 @@ def latent_decode_splits(rows: int, num_heads: int, reach: int,
 def latent_decode(qa: torch.Tensor, pages: torch.Tensor, block_table: torch.Tensor,
                   request_of_row: torch.Tensor, positions: torch.Tensor, out: torch.Tensor,
                   partial: torch.Tensor, *, num_heads: int, rank: int, scale: float,
-                  window: int, rows: int, splits: int) -> bool:
+                  window: int, rows: int, splits: int,
+                  sink: torch.Tensor | None = None) -> bool:
     """:func:`latent_attention` for steps of single rows: one CTA per (row, share of its
     keys) serves every head, so a latent row leaves memory once. A head's result lands in the
     first ``rank`` of its ``out.shape[1] / num_heads`` columns. ``partial`` is float32 scratch
@@ -1062,13 +1087,14 @@ def latent_decode(qa: torch.Tensor, pages: torch.Tensor, block_table: torch.Tens
             rows > positions.shape[0] or \
             partial.numel() < rows * num_heads * splits * (rank + 2):
         raise BackendError(f"{op}: shapes do not fit")
+    _need_sink(op, sink, num_heads)
     global _launches
     status = library("latent_attention").ayk_latent_decode(
         _ptr(qa), c_int(qa.stride(0)), _ptr(pages), _ptr(block_table),
         c_int(block_table.stride(0)), _ptr(request_of_row), _ptr(positions), _ptr(partial),
         _ptr(out), c_int(out.stride(0)), c_int(out.shape[1] // num_heads), c_int(rows),
         c_int(num_heads), c_int(rank), c_int(key_dim - rank), c_int(page_size), c_float(scale),
-        c_int(window), c_int(splits), c_int(_TYPE[qa.dtype]), _stream())
+        c_int(window), _ptr(sink), c_int(splits), c_int(_TYPE[qa.dtype]), _stream())
     if status == -6:  # AYK_NOT_TAKEN
         _launches -= 1
         return False
@@ -1885,9 +1911,12 @@ def pooled_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tens
 def norm_add(x: torch.Tensor, weight: torch.Tensor, eps: float, dst: torch.Tensor, *,
              factor: float = 1.0, weight_offset: float = 0.0, copy: torch.Tensor | None = None,
              rows: int, next_weight: torch.Tensor | None = None, next_eps: float = 1e-6,
-             next_offset: float = 0.0, next_out: torch.Tensor | None = None) -> None:
+             next_offset: float = 0.0, next_out: torch.Tensor | None = None,
+             x_factor: float = 1.0, other: torch.Tensor | None = None,
+             other_factor: float = 1.0) -> None:
     """``dst += factor * x * rsqrt(mean(x^2) + eps) * (weight_offset + weight)`` over float32
-    rows; with ``copy`` (float32 or bfloat16 ``[N, width]``) the new ``dst`` is also written
+    rows; with ``other`` (float32 like ``x``) ``x`` stands for ``x_factor * x + other_factor *
+    other``; with ``copy`` (float32 or bfloat16 ``[N, width]``) the new ``dst`` is also written
     there, rounded once; with ``next_out`` (of ``copy``'s type when both are given) and
     ``next_weight`` the new ``dst`` also leaves normalised for the sublayer that follows:
     ``next_out = dst * rsqrt(mean(dst^2) + next_eps) * (next_offset + next_weight)``."""
@@ -1901,6 +1930,12 @@ def norm_add(x: torch.Tensor, weight: torch.Tensor, eps: float, dst: torch.Tenso
     if x.shape[1] != width or weight.shape[0] != width or rows > x.shape[0] or \
             rows > dst.shape[0]:
         raise BackendError(f"{op}: shapes do not fit")
+    if other is not None:
+        _need(op, "other", other, torch.float32, 2)
+        if other.shape[1] != width or rows > other.shape[0]:
+            raise BackendError(f"{op}: other does not match x")
+    elif x_factor != 1.0:
+        raise BackendError(f"{op}: x_factor goes with other")
     if copy is not None:
         _need(op, "copy", copy, ndim=2)
         if copy.dtype not in _TYPE or copy.shape[1] != width or rows > copy.shape[0]:
@@ -1915,7 +1950,8 @@ def norm_add(x: torch.Tensor, weight: torch.Tensor, eps: float, dst: torch.Tenso
             raise BackendError(f"{op}: the next norm's output does not match dst")
         typed = next_out
     status = library("rms_norm").ayk_norm_add_next(
-        _ptr(x), c_int(x.stride(0)), _ptr(weight), c_float(weight_offset), c_float(eps),
+        _ptr(x), c_int(x.stride(0)), c_float(x_factor), _ptr(other),
+        c_int(0 if other is None else other.stride(0)), c_float(other_factor), _ptr(weight), c_float(weight_offset), c_float(eps),
         c_float(factor), _ptr(dst), c_int(dst.stride(0)), _ptr(copy),
         c_int(0 if copy is None else copy.stride(0)),
         c_int(0 if typed is None else _TYPE[typed.dtype]),
@@ -1934,12 +1970,13 @@ def gated_attention_prepare(proj: torch.Tensor, *, k_offset: int, v_offset: int,
                             k_pages: torch.Tensor | None, v_pages: torch.Tensor | None,
                             q: torch.Tensor, heads: int, kv_heads: int, dim: int, vdim: int,
                             rows: int, positions: torch.Tensor | None = None,
-                            freq: torch.Tensor | None = None, layout: str = "neighbours"
-                            ) -> None:
+                            freq: torch.Tensor | None = None, layout: str = "neighbours",
+                            head_norm: bool = False) -> None:
     """From a row of a fused projection (float32: ``heads * dim`` queries at 0, ``kv_heads *
     dim`` keys at ``k_offset``, ``kv_heads * vdim`` values at ``v_offset``): queries and keys
     each normalised by the root mean square over their whole projection with a weight per
-    entry (``None``: no norm), the first ``2 * len(freq)`` entries of every head rotated by the
+    entry (``None``: no norm), or with ``head_norm`` every head by its own root mean square with
+    one weight of ``dim`` entries for all heads, the first ``2 * len(freq)`` entries of every head rotated by the
     row's position (``freq`` ``None``: no rotation; see :func:`rope`), the queries written to ``q`` ``[N, heads * dim]``, the key and
     value into the row's cache slot (``k_pages`` ``[page, kv_head, slot, dim]``, ``v_pages``
     likewise with ``vdim``; ``None``: stored nowhere)."""
@@ -1950,8 +1987,8 @@ def gated_attention_prepare(proj: torch.Tensor, *, k_offset: int, v_offset: int,
     _need(op, "q", q, ndim=2)
     if q.dtype not in _TYPE:
         raise BackendError(f"{op}: float32 or bfloat16 only")
-    for name, tensor, size in (("q_weight", q_weight, heads * dim),
-                               ("k_weight", k_weight, kv_heads * dim)):
+    for name, tensor, size in (("q_weight", q_weight, dim if head_norm else heads * dim),
+                               ("k_weight", k_weight, dim if head_norm else kv_heads * dim)):
         if tensor is not None:
             _need(op, name, tensor, torch.float32)
             if tensor.numel() != size or not tensor.is_contiguous():
@@ -1984,20 +2021,43 @@ def gated_attention_prepare(proj: torch.Tensor, *, k_offset: int, v_offset: int,
         _ptr(k_pages), _ptr(v_pages), c_int(page_size), _ptr(q), c_int(q.stride(0)),
         c_int(rows), c_int(heads), c_int(kv_heads), c_int(dim), c_int(vdim),
         _ptr(positions if rot_dims else None), _ptr(freq if rot_dims else None),
-        c_int(rot_dims), c_int(ROPE_LAYOUTS[layout]), c_int(_TYPE[q.dtype]), _stream())
+        c_int(rot_dims), c_int(ROPE_LAYOUTS[layout]), c_int(1 if head_norm else 0),
+        c_int(_TYPE[q.dtype]), _stream())
     check(status, op)
+
+
+#: how the scores of :func:`gated_attention` become weights
+SCORES = ("softmax", "sigmoid")
+
+
+def _need_scores(op: str, scores: str, slope: torch.Tensor | None,
+                 score_bias: torch.Tensor | None, heads: int) -> int:
+    """The kernels' number for the way scores become weights (0: a plain softmax, 1: with
+    slopes, 2: a sigmoid), after a look at its vectors."""
+    if scores not in SCORES or (score_bias is not None and scores != "sigmoid"):
+        raise BackendError(f"{op}: scores are one of {SCORES}; a bias goes with a sigmoid")
+    for name, tensor in (("slope", slope), ("score_bias", score_bias)):
+        if tensor is not None:
+            _need(op, name, tensor, torch.float32, 1)
+            if tensor.shape[0] != heads:
+                raise BackendError(f"{op}: {name} has one entry per head")
+    return 2 if scores == "sigmoid" else (0 if slope is None else 1)
 
 
 def gated_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor,
                     block_table: torch.Tensor, request_of_row: torch.Tensor,
                     positions: torch.Tensor, out: torch.Tensor, *, heads: int, scale: float,
                     window: int = 0, keep_first: int = 0, gate: torch.Tensor | None = None,
-                    rows: int | None = None, tensor_cores: bool = True) -> None:
-    """Softmax attention over paged keys (``[page, kv_head, slot, dim]``) and values (``[...,
+                    rows: int | None = None, tensor_cores: bool = True,
+                    scores: str = "softmax", slope: torch.Tensor | None = None,
+                    score_bias: torch.Tensor | None = None) -> None:
+    """Attention over paged keys (``[page, kv_head, slot, dim]``) and values (``[...,
     vdim]``): the row of request ``request_of_row[i]`` at ``positions[i]`` sees key ``j <= p``
     when ``p - j < window`` (``window`` 0: always) or ``j < keep_first``; head ``h`` uses
-    key/value head ``h // (heads / kv_heads)``; scores ``scale * q . k`` and the softmax in
-    fp32; with ``gate`` (float32 ``[N, heads * vdim]``) the result is multiplied entry by
+    key/value head ``h // (heads / kv_heads)``; scores ``scale * q . k``, with ``slope`` (float32
+    ``[heads]``) less ``slope[h] * (p - j)``; weights in fp32: ``scores="softmax"`` over the
+    visible keys, or ``scores="sigmoid"``: each visible key's own ``sigmoid(score +
+    score_bias[h])`` (``score_bias`` float32 ``[heads]``, optional); with ``gate`` (float32 ``[N, heads * vdim]``) the result is multiplied entry by
     entry by ``sigmoid(gate)``. The step's own keys must already be stored."""
     op = "gated_attention"
     if _left_out and op in _left_out:
@@ -2027,8 +2087,9 @@ def gated_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tenso
         c_int(block_table.stride(0)), _ptr(request_of_row), _ptr(positions), _ptr(gate),
         c_int(0 if gate is None else gate.stride(0)), _ptr(out), c_int(out.stride(0)), c_int(n),
         c_int(heads), c_int(kv_heads), c_int(dim), c_int(vdim), c_int(page_size),
-        c_float(scale), c_int(window), c_int(keep_first), c_int(1 if tensor_cores else 0),
-        c_int(_TYPE[q.dtype]), _stream())
+        c_float(scale), c_int(window), c_int(keep_first),
+        c_int(_need_scores(op, scores, slope, score_bias, heads)), _ptr(slope),
+        _ptr(score_bias), c_int(1 if tensor_cores else 0), c_int(_TYPE[q.dtype]), _stream())
     check(status, op)
 
 
@@ -2045,7 +2106,9 @@ def gated_decode(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor,
                  block_table: torch.Tensor, request_of_row: torch.Tensor,
                  positions: torch.Tensor, out: torch.Tensor, partial: torch.Tensor | None, *,
                  heads: int, scale: float, window: int = 0, keep_first: int = 0,
-                 gate: torch.Tensor | None = None, rows: int, shares: int) -> bool:
+                 gate: torch.Tensor | None = None, rows: int, shares: int,
+                 scores: str = "softmax", slope: torch.Tensor | None = None,
+                 score_bias: torch.Tensor | None = None) -> bool:
     """:func:`gated_attention` for steps of single rows: a row's visible keys are cut into
     ``shares`` shares, one CTA each per head, and joined in their order. ``partial`` is
     float32 scratch of at least ``rows * heads * shares * (vdim + 2)`` elements (``None`` with
@@ -2081,6 +2144,7 @@ def gated_decode(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor,
         _need(op, "gate", gate, torch.float32, 2)
         if gate.shape[1] != heads * vdim or gate.shape[0] < rows or gate.stride(1) != 1:
             raise BackendError(f"{op}: the gate does not match the rows")
+    mode = _need_scores(op, scores, slope, score_bias, heads)
     global _launches
     status = library("gated_attention").ayk_gated_decode(
         _ptr(q), c_int(q.stride(0)), _ptr(k_pages), _ptr(v_pages), _ptr(block_table),
@@ -2088,7 +2152,8 @@ def gated_decode(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor,
         c_int(0 if gate is None else gate.stride(0)), _ptr(partial if shares > 1 else None),
         _ptr(out), c_int(out.stride(0)), c_int(rows), c_int(heads), c_int(kv_heads),
         c_int(dim), c_int(vdim), c_int(page_size), c_float(scale), c_int(window),
-        c_int(keep_first), c_int(shares), c_int(_TYPE[q.dtype]), _stream())
+        c_int(keep_first), c_int(mode), _ptr(slope), _ptr(score_bias), c_int(shares),
+        c_int(_TYPE[q.dtype]), _stream())
     if status == -6:  # AYK_NOT_TAKEN
         _launches -= 1
         return False

@@ -80,6 +80,7 @@ def architecture_of(config_json: Mapping[str, object]) -> Architecture:
 def _builtin() -> None:
     import ayaka_b200.models.gpt2  # noqa: F401  (registers itself)
     import ayaka_b200.models.gagotar  # noqa: F401
+    import ayaka_b200.models.kakilorn  # noqa: F401
     import ayaka_b200.models.mapuvik  # noqa: F401
     import ayaka_b200.models.rizitar  # noqa: F401
     import ayaka_b200.models.semadra  # noqa: F401

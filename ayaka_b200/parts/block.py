@@ -200,7 +200,9 @@ class OutputNormBlock(Block):
     in one scratch tensor that every kernel which updates the stream also refreshes
     (``ops.norm_add`` with ``copy``), so only a model's first layer pays a pass of its own for
     it. In float32 the sublayers read the stream directly. A sublayer writes into a scratch
-    branch (``forward_into`` where the part has it, else a zeroed branch it adds into)."""
+    branch (``forward_into`` where the part has it, else a zeroed branch it adds into); a mixer of
+    two sides with a factor each hands over both (``forward_branches``), and the norm's launch
+    joins them."""
 
     def __init__(self, spec: LayerSpec, ctx: BuildContext, position: Part | None) -> None:
         super().__init__(ctx)
@@ -218,6 +220,8 @@ class OutputNormBlock(Block):
             "side", build_part("side", spec.side.kind, spec.side, ctx))
         self.width = int(spec.mixer_norm.width)  # type: ignore[arg-type]
         self.factor = float(spec.residual_factor)
+        self.joins_sides = hasattr(self.mixer, "forward_branches") and \
+            len(getattr(self.mixer, "sides", ())) == 2
         for norm in (self.mixer_norm, self.feed_forward_norm):
             if norm is not None and not hasattr(norm, "add_normed"):
                 raise ValueError("an output_norm block needs norms that can add their result "
@@ -235,13 +239,19 @@ class OutputNormBlock(Block):
             stream = residual
         copy = stream if rounded else None
         branch = work.buffer("block.branch", self.width, torch.float32)
-        if hasattr(self.mixer, "forward_into"):
+        joined: dict[str, object] = {}
+        sides = self.mixer.forward_branches(stream, step, cache) \
+            if self.joins_sides else None  # type: ignore[attr-defined]
+        if sides is not None:
+            (first, x_factor), (other, other_factor) = sides
+            joined = dict(x_factor=x_factor, other=other, other_factor=other_factor)
+        elif hasattr(self.mixer, "forward_into"):
             self.mixer.forward_into(stream, branch, step, cache)  # type: ignore[attr-defined]
         else:
             branch[:n].zero_()
             self.mixer.forward(stream, branch, step, cache)  # type: ignore[attr-defined]
-        self.mixer_norm.add_normed(branch, residual, factor=self.factor,  # type: ignore
-                                   count=n, copy=copy)
+        self.mixer_norm.add_normed(first if sides is not None else branch,  # type: ignore
+                                   residual, factor=self.factor, count=n, copy=copy, **joined)
         if self.feed_forward_norm is not None:
             if hasattr(self.feed_forward, "forward_into"):
                 self.feed_forward.forward_into(stream, branch, step)  # type: ignore

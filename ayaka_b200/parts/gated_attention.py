@@ -1,4 +1,5 @@
-"""Softmax attention with rotated heads, a window that keeps the first tokens, an output gate."""
+"""Attention with rotated heads, a window that keeps the first tokens, an output gate; its weights
+a softmax over the visible keys or a sigmoid of each key's own score."""
 
 from __future__ import annotations
 
@@ -15,24 +16,29 @@ __all__ = ["GatedAttention"]
 
 @register_part("mixer", "gated_attention")
 class GatedAttention(Mixer):
-    """Grouped softmax attention over paged keys and values.
+    """Grouped attention over paged keys and values.
 
     One fused projection gives queries (``num_heads x head_dim``), keys (``num_kv_heads x
     head_dim``), values (``num_kv_heads x value_dim``) and, with ``gate``, one raw gate per
     entry of the joined heads. With ``qk_norm`` the whole query projection and the whole key
     projection are each normalised by their root mean square (all heads at once, a plain weight
-    per entry). With ``rot_dims`` the first so many entries of every query and key head are
+    per entry); with ``qk_norm="head"`` every head by its own, with one weight of ``head_dim``
+    entries that the heads share. With ``rot_dims`` the first so many entries of every query and key head are
     rotated by the position (``rot_layout``, frequencies ``rot_base^(-2i/rot_dims) / rot_slowed``);
     without, the scores know no positions. Query head ``h`` uses key/value head
     ``h // (num_heads / num_kv_heads)``; ``score = scale * q . k``; the query at position ``p`` sees
     key ``j <= p`` when ``p - j < window`` (``window`` 0: every earlier key) or ``j < keep_first``:
-    the sequence's first tokens stay in sight at their true positions; softmax in fp32; with
-    ``gate`` the joined heads are multiplied entry by entry by its sigmoid; then the output
+    the sequence's first tokens stay in sight at their true positions. With ``slopes`` (one number
+    per query head) ``slopes[h] * (p - j)`` is taken off the score, for a kept token too. The
+    weights, in fp32, are a softmax over the visible keys, or with ``weights="sigmoid"`` each key's
+    own ``sigmoid(score + b_h)`` (``score_bias``: the learned ``b``, one per head), which are not
+    normalised over the keys. With ``gate`` the joined heads are multiplied entry by entry by its sigmoid; then the output
     projection.
 
     Spec parameters: ``width``, ``num_heads``, ``num_kv_heads``, ``head_dim``, ``value_dim``,
-    ``scale``, ``window``, ``keep_first``, ``qk_norm``, ``eps``, ``gate``, ``rot_dims``,
-    ``rot_base``, ``rot_slowed``, ``rot_layout``.
+    ``scale``, ``window``, ``keep_first``, ``qk_norm`` (false, true or ``"head"``), ``eps``,
+    ``gate``, ``rot_dims``, ``rot_base``, ``rot_slowed``, ``rot_layout``, ``weights`` (``softmax``
+    or ``sigmoid``), ``score_bias``, ``slopes`` (a tuple).
     """
 
     def __init__(self, spec: PartSpec, ctx: BuildContext, position: Part | None = None) -> None:
@@ -65,9 +71,23 @@ class GatedAttention(Mixer):
         out_features = self.qkv_width + (self.out_width if self.gated else 0)
         self.proj_weight = self.add_param("proj.weight", (out_features, self.width), "matrix")
         self.q_norm = self.k_norm = None
+        self.head_norm = spec.get("qk_norm", False) == "head"
         if spec.get("qk_norm", False):
-            self.q_norm = self.add_param("q_norm.weight", (self.q_width,), "vector")
-            self.k_norm = self.add_param("k_norm.weight", (self.k_width,), "vector")
+            shared = dim if self.head_norm else 0
+            self.q_norm = self.add_param("q_norm.weight", (shared or self.q_width,), "vector")
+            self.k_norm = self.add_param("k_norm.weight", (shared or self.k_width,), "vector")
+        weights = str(spec.get("weights", "softmax"))
+        if weights not in ops.SCORES or (spec.get("score_bias", False) and weights != "sigmoid"):
+            raise ValueError(f"weights is one of {ops.SCORES}; a score_bias goes with sigmoid")
+        slopes = spec.get("slopes")
+        if slopes is not None and len(tuple(slopes)) != heads:  # type: ignore[arg-type]
+            raise ValueError(f"slopes has one number per query head ({heads})")
+        self.scoring: dict[str, object] = {
+            "scores": weights,
+            "slope": None if slopes is None else torch.tensor(
+                tuple(slopes), dtype=torch.float32, device=ctx.device),  # type: ignore[arg-type]
+            "score_bias": self.add_param("score_bias", (heads,), "vector")
+            if spec.get("score_bias", False) else None}
         self.out_weight = self.add_param("out.weight", (self.width, self.out_width), "matrix")
 
     def cache_need(self) -> CacheNeed:
@@ -101,10 +121,12 @@ class GatedAttention(Mixer):
             slot_mapping=group.slot_mapping, k_pages=cache.k_pages if cache.writes else None,
             v_pages=cache.v_pages if cache.writes else None, q=q, heads=self.num_heads,
             kv_heads=self.num_kv_heads, dim=self.head_dim, vdim=self.value_dim, rows=n,
-            positions=step.positions, freq=self._freq, layout=self.rot_layout)
+            positions=step.positions, freq=self._freq, layout=self.rot_layout,
+            head_norm=self.head_norm)
         gate = proj[:, self.qkv_width:] if self.gated else None
         # Prompt portions in bfloat16, where the sizes are the tensor-core kernel's: the
-        # engine's flash kernel, told of the kept keys, the value size and the gate. Single
+        # engine's flash kernel, told of the kept keys, the value size, the gate and the way
+        # scores become weights. Single
         # rows (a decode step, or the decoding requests that lead a mixed step) and every
         # other size or type go to this part's own kernel.
         tiled = dtype == torch.bfloat16 and not step.decode_only and \
@@ -125,18 +147,19 @@ class GatedAttention(Mixer):
                     q, cache.k_pages, cache.v_pages, group.block_table, step.request_of_row,
                     step.positions, attended, partial, heads=self.num_heads, scale=self.scale,
                     window=self.window, keep_first=self.keep_first, gate=gate, rows=lead,
-                    shares=shares):
+                    shares=shares, **self.scoring):
                 lead, taken = 0, lead
         if lead:
             ops.gated_attention(
                 q, cache.k_pages, cache.v_pages, group.block_table, step.request_of_row,
                 step.positions, attended, heads=self.num_heads, scale=self.scale,
-                window=self.window, keep_first=self.keep_first, gate=gate, rows=lead)
+                window=self.window, keep_first=self.keep_first, gate=gate, rows=lead,
+                **self.scoring)
         lead = lead or taken
         if tiled:
             ops.attention_prefill(
                 q, cache.k_pages, cache.v_pages, group.block_table[lead:],
                 step.row_start[lead:], step.kv_len[lead:], attended, num_heads=self.num_heads,
                 scale=self.scale, host_rows=step.host_rows[lead:], window=self.window,
-                keep_first=self.keep_first, gate=gate)
+                keep_first=self.keep_first, gate=gate, **self.scoring)
         ops.linear(attended, self.out_weight, None, out, residual=accumulate, rows=n)

@@ -6,8 +6,9 @@ import torch
 
 from ayaka_b200.kernels import ops
 from ayaka_b200.parts.base import BuildContext, CacheNeed, Part, register_part
-from ayaka_b200.parts.context import LayerCache, StepContext
-from ayaka_b200.parts.mixer import Mixer, attend_paged
+from ayaka_b200.parts.context import GroupStep, LayerCache, StepContext
+from ayaka_b200.parts.frequencies import blended_frequencies
+from ayaka_b200.parts.mixer import Mixer, attend_paged, leading_single_rows
 from ayaka_b200.parts.spec import PartSpec
 
 __all__ = ["LatentAttention"]
@@ -41,11 +42,15 @@ class LatentAttention(Mixer):
     output gate out; ``shares_latent=True`` is a layer without a down-projection of its own:
     it reads the latent rows another run of the order stored (``Run.reads_cache_of``) with its
     own up-projections, queries and window. ``rot`` may be 0 (no positions in the scores).
+    ``gate="head"``: one gate per head instead of one per entry of the joined heads.
+    ``rot_scaling`` (factor, original, fast, slow): frequencies and gain of
+    :func:`~ayaka_b200.parts.frequencies.blended_frequencies`. ``sink``: the softmax's denominator
+    also holds ``exp(sink_h)``, one learned number per head.
 
     Spec parameters: ``width``, ``num_heads``, ``dim``, ``rot``, ``value_dim``, ``rank``,
     ``scale``, ``window`` (0 = none), ``rot_dims``, ``rot_base``, ``rot_layout``
-    (``neighbours`` when absent), ``eps`` (of the norms), ``query_rank`` (0 when absent),
-    ``gate`` (true when absent), ``shares_latent`` (false when absent).
+    (``neighbours`` when absent), ``rot_scaling``, ``eps`` (of the norms), ``query_rank`` (0 when
+    absent), ``gate`` (true when absent), ``shares_latent``, ``sink`` (false when absent).
     """
 
     def __init__(self, spec: PartSpec, ctx: BuildContext, position: Part | None = None) -> None:
@@ -64,6 +69,8 @@ class LatentAttention(Mixer):
         self.eps = float(spec.eps)  # type: ignore[arg-type]
         self.query_rank = int(spec.get("query_rank", 0))  # type: ignore[arg-type]
         self.gated = bool(spec.get("gate", True))
+        self.rot_scaling = spec.get("rot_scaling")
+        self.rot_gain = 1.0
         self.shares_latent = bool(spec.get("shares_latent", False))
         if self.rot_dims % 2 or not 0 <= self.rot_dims <= self.rot:
             raise ValueError(f"rot_dims must be even and at most rot ({self.rot}), got "
@@ -80,7 +87,9 @@ class LatentAttention(Mixer):
         first = self.query_rank or self.q_width
         self.kv_offset = self.q_width + self.query_rank
         self.gate_offset = self.kv_offset + own
-        rows = first + own + (self.out_width if self.gated else 0)
+        gates = self.num_heads if spec.get("gate", True) == "head" else self.out_width
+        self.gate_width = gates if self.gated else 0
+        rows = first + own + self.gate_width
         self.proj_weight = self.add_param("proj.weight", (rows, self.width), "matrix")
         self.q_norm = self.q_up = None
         if self.query_rank:
@@ -91,6 +100,8 @@ class LatentAttention(Mixer):
         self.up_key = self.add_param("up_key.weight", (self.num_heads * self.dim, self.rank),
                                      "matrix")
         self.up_value = self.add_param("up_value.weight", (self.out_width, self.rank), "matrix")
+        self.sink = self.add_param("sink", (self.num_heads,), "vector") \
+            if spec.get("sink", False) else None
         self.out_weight = self.add_param("out.weight", (self.width, self.out_width), "matrix")
         self._freq: torch.Tensor | None = None
         self._no_weight: torch.Tensor | None = None
@@ -112,7 +123,7 @@ class LatentAttention(Mixer):
         n, dtype, work = step.num_rows, self.ctx.dtype, step.workspace
         heads, rank = self.num_heads, self.rank
         if self._freq is None:
-            self._freq = ops.rope_frequencies(max(self.rot_dims, 0), self.rot_base, hidden.device)
+            self._freq = self._frequencies(hidden.device)
             self._no_weight = torch.ones(rank, dtype=torch.float32, device=hidden.device)
         if cache.writes == self.shares_latent:
             raise ValueError("a latent attention layer either stores its latents or reads "
@@ -142,31 +153,58 @@ class LatentAttention(Mixer):
             eps=self.eps, positions=step.positions, slot_mapping=group.slot_mapping,
             freq=self._freq, layout=self.rot_layout,
             pages=cache.k_pages if cache.writes else None,
-            q_plain=q_plain, qa=qa, heads=heads, dim=self.dim, rot=self.rot, rank=rank, rows=n)
+            q_plain=q_plain, qa=qa, heads=heads, dim=self.dim, rot=self.rot, rank=rank, rows=n,
+            rot_gain=self.rot_gain)
         # the queries' unrotated parts, taken to latent space: qa[:, h, :rank] = W_uk,h^T q
         ops.head_linear(q_plain, self.up_key, qa, heads=heads, transposed=True, rows=n)
-        taken = False
-        if step.decode_only:
-            # single rows: the kernel that fetches a latent row once for all heads
-            reach = min(step.max_kv_len, self.window) if self.window else step.max_kv_len
-            splits = ops.latent_decode_splits(n, heads, reach, hidden.device)
-            partial = work.buffer("latent.partial", heads * (rank + 2), torch.float32,
-                                  rows=n * splits)
-            taken = ops.latent_decode(qa, cache.k_pages, group.block_table,
-                                      step.request_of_row, step.positions, mixed, partial,
-                                      num_heads=heads, rank=rank, scale=self.scale,
-                                      window=self.window, rows=n, splits=splits)
-        if taken:
-            pass
-        elif shared:
-            attend_paged(qa, cache.k_pages, cache.k_pages, mixed, step, group, num_heads=heads,
-                         scale=self.scale, window=self.window, dtype=dtype)
-        else:
-            ops.latent_attention(qa, cache.k_pages, group.block_table, step.request_of_row,
-                                 step.positions, mixed, num_heads=heads, rank=rank,
-                                 scale=self.scale, window=self.window, rows=n)
-        gate = proj[:, self.gate_offset:self.gate_offset + self.out_width] if self.gated \
+        self._attend(qa, mixed, step, cache, group, shared)
+        gate = proj[:, self.gate_offset:self.gate_offset + self.gate_width] if self.gated \
             else None
         ops.head_linear(mixed, self.up_value, attended, heads=heads, transposed=False, rows=n,
                         gate=gate, inner=rank)
         ops.linear(attended, self.out_weight, None, residual, residual=accumulate, rows=n)
+
+    def _frequencies(self, device: torch.device) -> torch.Tensor:
+        if self.rot_scaling is None or not self.rot_dims:
+            return ops.rope_frequencies(self.rot_dims, self.rot_base, device)
+        factor, original, fast, slow = (float(v) for v in self.rot_scaling)  # type: ignore
+        values, self.rot_gain = blended_frequencies(
+            self.rot_dims, self.rot_base, factor=factor, original=original, fast=fast, slow=slow)
+        return torch.tensor(values, dtype=torch.float64, device=device)
+
+    def _attend(self, qa: torch.Tensor, mixed: torch.Tensor, step: StepContext,
+                cache: LayerCache, group: GroupStep, shared: bool) -> None:
+        """Weighted sums of the latent rows. Single rows (a decode step; with a sink also the
+        decoding requests that lead a mixed step) go to the kernel that fetches a latent row once
+        for all heads, portions to the engine's attention kernels when the rows are a head size
+        of theirs (``shared``), what is left to the generic kernel."""
+        n, heads, rank = step.num_rows, self.num_heads, self.rank
+        tiled = shared and self.ctx.dtype == torch.bfloat16 and not step.decode_only
+        lead = n if step.decode_only else 0
+        if tiled and self.sink is not None:
+            lead = leading_single_rows(step.host_rows)
+        if lead:
+            reach = min(step.max_kv_len, self.window) if self.window else step.max_kv_len
+            splits = ops.latent_decode_splits(lead, heads, reach, qa.device)
+            partial = step.workspace.buffer("latent.partial", heads * (rank + 2), torch.float32,
+                                            rows=n * splits)
+            if not ops.latent_decode(qa, cache.k_pages, group.block_table, step.request_of_row,
+                                     step.positions, mixed, partial, num_heads=heads, rank=rank,
+                                     scale=self.scale, window=self.window, rows=lead,
+                                     splits=splits, sink=self.sink):
+                lead, tiled = 0, False
+        if lead == n:
+            return
+        if shared and self.sink is None:
+            attend_paged(qa, cache.k_pages, cache.k_pages, mixed, step, group, num_heads=heads,
+                         scale=self.scale, window=self.window, dtype=self.ctx.dtype)
+        elif tiled:
+            ops.attention_prefill(
+                qa, cache.k_pages, cache.k_pages, group.block_table[lead:],
+                step.row_start[lead:], step.kv_len[lead:], mixed, num_heads=heads,
+                scale=self.scale, host_rows=step.host_rows[lead:], window=self.window,
+                sink=self.sink)
+        else:
+            ops.latent_attention(qa, cache.k_pages, group.block_table, step.request_of_row,
+                                 step.positions, mixed, num_heads=heads, rank=rank,
+                                 scale=self.scale, window=self.window, rows=n, sink=self.sink)

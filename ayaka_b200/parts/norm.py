@@ -71,16 +71,19 @@ class RMSNorm(Part):
 
     def add_normed(self, x: torch.Tensor, residual: torch.Tensor, *, factor: float, count: int,
                    copy: torch.Tensor | None = None, then: RMSNorm | None = None,
-                   then_out: torch.Tensor | None = None) -> None:
+                   then_out: torch.Tensor | None = None, x_factor: float = 1.0,
+                   other: torch.Tensor | None = None, other_factor: float = 1.0) -> None:
         """``residual += factor * norm(x)`` over ``count`` fp32 rows (a norm on a sublayer's
-        *output*); with ``copy`` the new rows of the stream are also written there in its
+        *output*; with ``other``, of ``x_factor * x + other_factor * other``); with ``copy`` the new rows of the stream are also written there in its
         type, for the sublayer that reads them next; with ``then`` (the norm in front of the
         next sublayer) and ``then_out`` that norm's output leaves the same launch."""
+        joined = {} if other is None else dict(x_factor=x_factor, other=other,
+                                               other_factor=other_factor)
         if then is None or then_out is None:
             ops.norm_add(x, self.weight, self.eps, residual, factor=factor,
-                         weight_offset=self.offset, copy=copy, rows=count)
+                         weight_offset=self.offset, copy=copy, rows=count, **joined)
         else:
             ops.norm_add(x, self.weight, self.eps, residual, factor=factor,
                          weight_offset=self.offset, copy=copy, rows=count,
                          next_weight=then.weight, next_eps=then.eps, next_offset=then.offset,
-                         next_out=then_out)
+                         next_out=then_out, **joined)

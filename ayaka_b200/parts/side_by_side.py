@@ -17,17 +17,22 @@ __all__ = ["SideBySide", "TalkingAttention"]
 
 @register_part("mixer", "side_by_side")
 class SideBySide(Mixer):
-    """Several mixers read the same normed input; each result is normalised over the model's
-    width by its root mean square with a weight of its own, and the mixer returns their mean:
+    """Several mixers read the same input. Each result is normalised over the model's width by its
+    root mean square with a weight of its own, and the mixer returns their mean:
     ``(1 / n) * sum_b rms(side_b(h)) * w_b``. The join, an optional scale of the layer and the
     sum into the residual stream are one kernel (``ops.norm_sum``).
+
+    With ``scales`` (a number per side) nothing is normalised: the mixer returns
+    ``sum_b scales[b] * side_b(h)``. A block that norms a mixer's result asks for the two sides and
+    their scales instead (``forward_branches``) and joins them in its norm's launch.
 
     At most one side may keep pages and at most one a per-request state (a layer has one
     cache and one state). A side that has ``forward_into(hidden, out, step, cache)`` writes
     its result into its scratch rows; any other mixer adds into zeroed rows.
 
     Spec parameters: ``width``, ``eps``, ``sides`` (a tuple of mixer ``PartSpec``), ``names``
-    (the sides' names: children ``<name>`` and parameters ``<name>_out.weight``).
+    (the sides' names: children ``<name>`` and, without ``scales``, parameters
+    ``<name>_out.weight``), ``scales``.
     """
 
     def __init__(self, spec: PartSpec, ctx: BuildContext, position: Part | None = None) -> None:
@@ -38,12 +43,19 @@ class SideBySide(Mixer):
         names = tuple(spec.names)  # type: ignore[arg-type]
         if not 1 <= len(sides) <= 4 or len(names) != len(sides) or len(set(names)) != len(names):
             raise ValueError("side_by_side takes one to four sides with a name each")
+        scales = spec.get("scales")
+        self.scales = None if scales is None else tuple(float(s) for s in scales)  # type: ignore
+        if self.scales is not None and len(self.scales) != len(sides):
+            raise ValueError("scales has one number per side")
+        self._scale_rows: list[torch.Tensor] = []
         self.sides: list[Mixer] = []
         self.weights: list[torch.Tensor] = []
         for name, side in zip(names, sides):
             part = build_part("mixer", side.kind, side, ctx, position)
             self.sides.append(self.add_child(str(name), part))  # type: ignore[arg-type]
-            self.weights.append(self.add_param(f"{name}_out.weight", (self.width,), "vector"))
+            if self.scales is None:
+                self.weights.append(self.add_param(f"{name}_out.weight", (self.width,),
+                                                   "vector"))
         if sum(side.cache_need() is not None for side in self.sides) > 1 or \
                 sum(side.state_need() is not None for side in self.sides) > 1:
             raise ValueError("at most one side may keep pages and at most one a state")
@@ -60,15 +72,44 @@ class SideBySide(Mixer):
                 cache: LayerCache) -> None:
         self.forward_scaled(hidden, residual, step, cache, None)
 
-    #: ``forward_scaled`` takes ``then``: a root-mean-square norm that its last kernel applies
-    #: to the rows of the stream it has updated
-    applies_next_norm = True
+    @property
+    def applies_next_norm(self) -> bool:
+        """Whether ``forward_scaled`` takes ``then``: a root-mean-square norm that its last kernel
+        applies to the rows of the stream it has updated."""
+        return self.scales is None
 
     def forward_scaled(self, hidden: torch.Tensor, residual: torch.Tensor, step: StepContext,
                        cache: LayerCache, scale: torch.Tensor | None,
                        then: Part | None = None, then_out: torch.Tensor | None = None) -> None:
         n = step.num_rows
-        branches = []
+        branches = self._branches(hidden, step, cache)
+        if self.scales is not None:
+            if scale is not None or then is not None:
+                raise ValueError("sides with scales take no scale of the layer and no next norm")
+            for branch, row in zip(branches, self._constant_rows(hidden.device)):
+                ops.scale_add(branch, row, residual, rows=n)
+            return
+        following = {} if then is None else then.as_next(then_out)  # type: ignore
+        ops.norm_sum(branches, self.weights, self.eps, residual, factor=1.0 / len(branches),
+                     scale=scale, accumulate=True, rows=n, **following)
+
+    def forward_branches(self, hidden: torch.Tensor, step: StepContext,
+                         cache: LayerCache) -> list[tuple[torch.Tensor, float]] | None:
+        """The sides' results (fp32 scratch rows) with the numbers they are multiplied by, or
+        ``None``, having run nothing, when the result is not such a sum."""
+        if self.scales is None:
+            return None
+        return list(zip(self._branches(hidden, step, cache), self.scales))
+
+    def _constant_rows(self, device: torch.device) -> list[torch.Tensor]:
+        if not self._scale_rows:
+            self._scale_rows = [torch.full((self.width,), s, dtype=torch.float32, device=device)
+                                for s in self.scales or ()]
+        return self._scale_rows
+
+    def _branches(self, hidden: torch.Tensor, step: StepContext,
+                  cache: LayerCache) -> list[torch.Tensor]:
+        n, branches = step.num_rows, []
         for index, side in enumerate(self.sides):
             branch = step.workspace.buffer(f"side_by_side.{index}", self.width, torch.float32)
             if hasattr(side, "forward_into"):
@@ -77,9 +118,7 @@ class SideBySide(Mixer):
                 branch[:n].zero_()
                 side.forward(hidden, branch, step, cache)
             branches.append(branch)
-        following = {} if then is None else then.as_next(then_out)  # type: ignore
-        ops.norm_sum(branches, self.weights, self.eps, residual, factor=1.0 / len(branches),
-                     scale=scale, accumulate=True, rows=n, **following)
+        return branches
 
 
 @register_part("mixer", "talking_attention")
