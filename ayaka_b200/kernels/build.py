@@ -49,9 +49,12 @@ def _nvcc() -> str | None:
     return None
 
 
-#: Libraries compiled once per value of a macro, and the values :func:`build_all` prepares.
-VARIANTS: dict[str, tuple[str, tuple[int, ...]]] = {
-    "attention_prefill": ("AYK_HEAD_DIM", (16, 32, 48, 64, 128)),
+#: Libraries compiled once per set of macro values, and the sets :func:`build_all` prepares
+#: (others are compiled when a model first asks for them).
+VARIANTS: dict[str, tuple[dict[str, int], ...]] = {
+    "attention_prefill": (
+        *({"AYK_HEAD_DIM": dim} for dim in (16, 32, 48, 64, 128)),
+        *({"AYK_HEAD_DIM": 64, "AYK_SCORES": scores} for scores in (1, 2))),
 }
 
 
@@ -158,8 +161,7 @@ def build_all(*, verbose: bool = True) -> list[Path]:
     jobs: list[tuple[str, dict[str, int] | None]] = []
     for name in library_names():
         if name in VARIANTS:
-            macro, values = VARIANTS[name]
-            jobs.extend((name, {macro: value}) for value in values)
+            jobs.extend((name, defines) for defines in VARIANTS[name])
         else:
             jobs.append((name, None))
     with ThreadPoolExecutor(max_workers=max(1, min(os.cpu_count() or 1, len(jobs)))) as pool:

@@ -23,7 +23,8 @@ workloads of BASELINE.json's other configurations (see :func:`workload_run`);
 ``--design mapuvik`` runs that design beside GPT-2 of equal size, ``--design gagotar`` that
 design beside Mapuvik and GPT-2, ``--design semadra`` that design beside Gagotar, Mapuvik and
 GPT-2, ``--design rizitar`` that design beside Semadra, Gagotar and GPT-2, ``--design senurax``
-that design beside Rizitar, Semadra, Gagotar and GPT-2 (``bench_design.py``).
+that design beside Rizitar, Semadra, Gagotar and GPT-2, ``--design kakilorn`` that design beside
+Senurax, Semadra, Mapuvik and GPT-2 (``bench_design.py``).
 """
 
 from __future__ import annotations
@@ -521,11 +522,11 @@ def main() -> int:
                              "(GPT-2 small with 64 ragged requests; GPT-2 large with prompt "
                              "portions beside 32 decoding requests)")
     parser.add_argument("--design", choices=("mapuvik", "gagotar", "semadra", "rizitar",
-                                               "senurax"),
+                                               "senurax", "kakilorn"),
                         help="instead of the headline run: the named design beside GPT-2 (and, "
                              "for gagotar, Mapuvik; for semadra, Gagotar and Mapuvik; for "
-                             "rizitar and senurax, the designs with like kernels) of equal "
-                             "size, prompt step and decode step "
+                             "rizitar, senurax and kakilorn, the designs with like kernels) of "
+                             "equal size, prompt step and decode step "
                              "with per-kernel times (bench_design.py); --sizes picks among "
                              "1024,2048")
     parser.add_argument("--sizes", default=None, help="with --design: widths to run")

@@ -1,12 +1,14 @@
-"""``bench.py --design mapuvik`` / ``gagotar`` / ``semadra`` / ``rizitar`` / ``senurax``: prefill and
-decode throughput of the design at sizes that resemble a real model's layers, beside GPT-2 of the same
+"""``bench.py --design mapuvik`` / ``gagotar`` / ``semadra`` / ``rizitar`` / ``senurax`` / ``kakilorn``:
+prefill and decode throughput of the design at sizes that resemble a real model's layers, beside GPT-2 of the same
 width, heads, feed-forward and number of layers (Gagotar also beside Mapuvik, the design whose
 kernels are closest to its own; Semadra beside Gagotar, whose experts and attention, and
 Mapuvik, whose latent attention are the like kernels; Rizitar beside Semadra, whose windowed
 attention, norms behind the sublayers, experts and token input, and Gagotar, whose scan over a
 matrix state are the like kernels; Senurax beside Rizitar, whose delta rule, Semadra, whose
 attention and gated experts, and Gagotar, whose linear attention beside a softmax attention are
-the like kernels), on one B200 with random bf16 weights.
+the like kernels; Kakilorn beside Senurax, whose delta rules, Semadra, whose windowed attention,
+output norms and gated feed-forward, and Mapuvik, whose latent attention with a rotated part are the
+like kernels), on one B200 with random bf16 weights.
 
 For each size and model: one prompt step of 2,048 tokens (two prompts of 1,024) and one decode
 step of 8 requests at context 1,025, each timed on the device as a CUDA-graph replay of the
@@ -154,6 +156,30 @@ def senurax_config(width: int, heads: int, ff: int, repeats: int, vocab: int) ->
             "layers": [ends, *middle, ends]}
 
 
+#: Kakilorn at the bench's sizes: latent rows of 256 entries as in Mapuvik's configuration, the
+#: query latent, window and kept tokens of Semadra's, the delta rules of Senurax's; a gated dense
+#: feed-forward in every layer
+def kakilorn_config(width: int, heads: int, ff: int, repeats: int, vocab: int) -> dict:
+    head = width // heads
+    latent = {"heads": heads, "dim": head, "rot_dim": head // 2, "vdim": head,
+              "q_rank": width // 2, "kv_rank": 256 - head // 2,
+              "scale": (head + head // 2) ** -0.5,
+              "rot": {"base": 500000.0, "dims": head // 2,
+                      "scaling": {"factor": 4.0, "original": 8192, "fast": 32.0, "slow": 1.0}}}
+    delta = {"heads": width // 64, "kv_heads": width // 64, "dim": 64, "vdim": 64, "conv": 4}
+    left = {"heads": heads, "kv_heads": heads // 4, "dim": head, "vdim": head,
+            "scale": head ** -0.5,
+            "mask": {"size": SEMADRA_WINDOW, "keep_first": SEMADRA_KEEP}}
+    parallel = {"left": left, "right": delta, "left_scale": 0.5, "right_scale": 0.9}
+    channel = {**delta, "decay_rank": 64, "gate_rank": 64}
+    mlp = {"kind": "dense", "ff": ff}
+    layers = [{"type": kind, "mixer": mixer, "mlp": mlp} for _ in range(repeats)
+              for kind, mixer in (("latent_attention", latent), ("parallel", parallel),
+                                  ("channel_delta", channel))]
+    return {"architecture": "Kakilorn", "vocab": vocab, "width": width, "norm": {"eps": 1e-5},
+            "embedding": {"scale": width ** 0.5}, "logit_scale": 0.5, "layers": layers}
+
+
 def gpt2_config(width: int, heads: int, ff: int, layers: int, vocab: int) -> dict:
     return {"architectures": ["GPT2LMHeadModel"], "n_layer": layers, "n_embd": width,
             "n_head": heads, "n_inner": ff, "vocab_size": vocab, "n_positions": 2 * LENGTH,
@@ -249,32 +275,83 @@ def _class_work(config: dict, rows: int, keys_per_row: float, decode: bool,
             add("moe_join", 0.0, rows * width * (4 * top + 10))
         product(config["vocab"], width, 4, wanted)
         return work
+
+    def linear_attention(m: dict, decay: int, taps: int, channel: bool) -> None:
+        """A recurrence and what goes with it: ``decay`` raw decays a row."""
+        H, kv, N, P = m["heads"], m.get("kv_heads", m["heads"]), m["dim"], m["vdim"]
+        channels = 2 * kv * N + H * P
+        state = 2 * H * N * P * 4 * (rows if decode else PROMPTS)
+        if decode:  # one kernel: convolution, low-rank pairs, state, norm and gate
+            up = H * (N + P) * m["gate_rank"] * 2 if channel else 0
+            add("linear_attention_decode", 8.0 * rows * H * N * P,
+                rows * (channels * 4 * (1 + taps) + H * P * 6) + state + up)
+            return
+        if taps:
+            add("conv_ring", 2.0 * rows * channels * taps, rows * channels * 8)
+        if channel:
+            for rank, n in ((m["decay_rank"], H * N), (m["gate_rank"], H * P)):
+                add("cast_rows", 0.0, rows * rank * 6)
+                product(n, rank, 4)
+        add("linear_attention_chunks", 8.0 * rows * H * N * P,
+            rows * (channels + decay + H * P) * 4 + state)
+        add("rms_norm", 0.0, rows * H * P * 10)
+
+    def gated(inner: int) -> None:  # act(gate) * up between two products
+        product(2 * inner, width, 4)
+        add("gated_unit", 0.0, rows * inner * 10)
+        product(width, inner, 4)
+
+    if config["architecture"] == "Kakilorn":
+        add("cast_rows", 0.0, rows * width * 6)
+        reuse = 1 if decode else 64 / 8  # a tile of 64 rows shares its keys
+        for layer in config["layers"]:
+            m = layer["mixer"]
+            if layer["type"] == "latent_attention":
+                H, dim, rot, vdim = m["heads"], m["dim"], m["rot_dim"], m["vdim"]
+                rank, q_rank = m["kv_rank"], m["q_rank"]
+                product(q_rank + rank + rot + H, width, 4)
+                add("rms_norm", 0.0, rows * q_rank * 6)
+                product(H * (dim + rot), q_rank, 4)
+                add("latent_prepare", 0.0, rows * (H * (dim + rot) + rank + rot) * 6)
+                add("head_linear", 2.0 * rows * H * rank * (dim + vdim),
+                    H * rank * (dim + vdim) * 2 + rows * H * (dim + vdim + 2 * rank) * 2)
+                add("latent_attention", 2.0 * rows * keys_per_row * H * (2 * rank + rot),
+                    rows * keys_per_row * (rank + rot) * 2 / reuse)
+                product(width, H * vdim, 4)
+                add("norm_add", 0.0, rows * width * 14)
+            elif layer["type"] == "channel_delta":
+                H, kv, N, P = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+                product(2 * kv * N + H * P + m["decay_rank"] + m["gate_rank"] + H, width, 4)
+                linear_attention(m, H * N, m["conv"], True)
+                product(width, H * P, 4)
+                add("norm_add", 0.0, rows * width * 14)
+            else:
+                a, r = m["left"], m["right"]
+                H, G, dim, vdim = a["heads"], a["kv_heads"], a["dim"], a["vdim"]
+                window, keep = a["mask"]["size"], a["mask"]["keep_first"]
+                spans = [p + 1 if p < window else window + min(keep, p + 1 - window)
+                         for p in ([int(keys_per_row) - 1] if decode else range(LENGTH))]
+                keys = sum(spans) / len(spans)
+                product(H * dim + G * (dim + vdim), width, 4)
+                add("gated_attention_prepare", 0.0, rows * (H * dim + G * (dim + vdim)) * 6)
+                add("gated_attention", 2.0 * rows * keys * H * (dim + vdim),
+                    rows * keys * G * (dim + vdim) * 2 / reuse + rows * H * (dim + vdim) * 2)
+                product(width, H * vdim, 4)
+                H, kv, N, P = r["heads"], r["kv_heads"], r["dim"], r["vdim"]
+                product(2 * kv * N + 2 * H * P + 2 * H, width, 4)
+                linear_attention(r, H, r["conv"], False)
+                product(width, H * P, 4)
+                add("norm_add", 0.0, rows * width * 18)
+            gated(layer["mlp"]["ff"])
+            add("norm_add", 0.0, rows * width * 14)
+        add("rms_norm", 0.0, wanted * width * 6)
+        product(config["vocab"], width, 4, wanted)
+        return work
     if config["architecture"] == "Senurax":
         loop = config["loop"]
         layers = config["layers"]
         order = [*layers[:loop["start"]], *(layers[loop["start"]:loop["stop"]] * loop["times"]),
                  *layers[loop["stop"]:]]
-
-        def linear_attention(m: dict, decay: int, taps: int, channel: bool) -> None:
-            """A recurrence and what goes with it: ``decay`` raw decays a row."""
-            H, kv, N, P = m["heads"], m.get("kv_heads", m["heads"]), m["dim"], m["vdim"]
-            channels = 2 * kv * N + H * P
-            state = 2 * H * N * P * 4 * (rows if decode else PROMPTS)
-            if decode:  # one kernel: convolution, low-rank pairs, state, norm and gate
-                up = H * (N + P) * m["gate_rank"] * 2 if channel else 0
-                add("linear_attention_decode", 8.0 * rows * H * N * P,
-                    rows * (channels * 4 * (1 + taps) + H * P * 6) + state + up)
-                return
-            if taps:
-                add("conv_ring", 2.0 * rows * channels * taps, rows * channels * 8)
-            if channel:
-                for rank, n in ((m["decay_rank"], H * N), (m["gate_rank"], H * P)):
-                    add("cast_rows", 0.0, rows * rank * 6)
-                    product(n, rank, 4)
-            add("linear_attention_chunks", 8.0 * rows * H * N * P,
-                rows * (channels + decay + H * P) * 4 + state)
-            add("rms_norm", 0.0, rows * H * P * 10)
-
         add("cast_rows", 0.0, rows * width * 6 * (1 + loop["times"]))
         for _ in range(loop["times"]):
             product(width, 2 * width, 4)
@@ -394,12 +471,6 @@ def _class_work(config: dict, rows: int, keys_per_row: float, decode: bool,
     if config["architecture"] == "Semadra":
         side = (config.get("token_side") or {}).get("dim", 0)
         add("cast_rows", 0.0, rows * width * 6)
-
-        def gated(inner: int) -> None:  # act(gate) * up between two products
-            product(2 * inner, width, 4)
-            add("gated_unit", 0.0, rows * inner * 10)
-            product(width, inner, 4)
-
         for layer in config["layers"]:
             m, mlp = layer["mixer"], layer["mlp"]
             H, dim, vdim = m["heads"], m["dim"], m["vdim"]
@@ -642,13 +713,16 @@ def run(sizes: str | None = None, design: str = "mapuvik") -> dict:
     for name in picked:
         width, heads, ff, repeats = table[name]
         results[name] = {"layers": 3 * repeats, "width": width, "heads": heads, "ff": ff}
-        if design == "senurax":
+        if design == "kakilorn":
+            results[name]["kakilorn"] = _measure(
+                kakilorn_config(width, heads, ff, repeats, 32000), peak)
+        if design in ("senurax", "kakilorn"):
             results[name]["senurax"] = _measure(
                 senurax_config(width, heads, ff, repeats, 32000), peak)
         if design in ("rizitar", "senurax"):
             results[name]["rizitar"] = _measure(
                 rizitar_config(width, heads, ff, repeats, 32000), peak)
-        if design in ("semadra", "rizitar", "senurax"):
+        if design in ("semadra", "rizitar", "senurax", "kakilorn"):
             results[name]["semadra"] = _measure(
                 semadra_config(width, heads, ff, repeats, 32000), peak)
         if design in ("gagotar", "semadra", "rizitar", "senurax"):
@@ -658,7 +732,8 @@ def run(sizes: str | None = None, design: str = "mapuvik") -> dict:
             results[name]["mapuvik"] = _measure(
                 mapuvik_config(width, heads, ff, repeats, 32000), peak)
         results[name]["gpt2"] = _measure(gpt2_config(width, heads, ff, 3 * repeats, 32000), peak)
-    title = {"senurax": "Senurax beside Rizitar, Semadra, Gagotar and GPT-2",
+    title = {"kakilorn": "Kakilorn beside Senurax, Semadra, Mapuvik and GPT-2",
+             "senurax": "Senurax beside Rizitar, Semadra, Gagotar and GPT-2",
              "rizitar": "Rizitar beside Semadra, Gagotar and GPT-2",
              "gagotar": "Gagotar beside Mapuvik and GPT-2",
              "semadra": "Semadra beside Gagotar, Mapuvik and GPT-2"}.get(

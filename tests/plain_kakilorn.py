@@ -152,9 +152,11 @@ def rotary_frequencies(rot: dict) -> tuple[np.ndarray, float]:
     return f / factor * ramp + f * (1.0 - ramp), 0.1 * math.log(factor) + 1.0
 
 
-def rotate(x: np.ndarray, rot: dict) -> np.ndarray:
+def rotate(x: np.ndarray, rot: dict | None) -> np.ndarray:
     """``x`` ``[T, heads, n]``: entries ``2i`` and ``2i + 1`` of the first ``rot.dims`` turned
     by the position, seen as a complex number."""
+    if not rot:
+        return x
     dims = int(rot["dims"])
     f, gain = rotary_frequencies(rot)
     turn = gain * np.exp(1j * np.arange(x.shape[0])[:, None] * f[None, :])[:, None, :]
@@ -169,10 +171,10 @@ def latent_attention(h: np.ndarray, t: dict, p: str, mixer: dict, eps: float) ->
     rank, vdim, count = int(mixer["kv_rank"]), int(mixer["vdim"]), h.shape[0]
     q = rms(h @ t[p + "dq"].T, t[p + "dq.norm"], eps) @ t[p + "uq"].T
     q = q.reshape(count, heads, dim + rot_dim)
-    q_turned = rotate(q[..., dim:], mixer["rot"])
+    q_turned = rotate(q[..., dim:], mixer.get("rot"))
     down = h @ t[p + "dkv"].T
     c = rms(down[:, :rank], t[p + "dkv.norm"], eps)
-    k_turned = rotate(down[:, None, rank:], mixer["rot"])[:, 0]
+    k_turned = rotate(down[:, None, rank:], mixer.get("rot"))[:, 0]
     k = (c @ t[p + "uk"].T).reshape(count, heads, dim)
     v = (c @ t[p + "uv"].T).reshape(count, heads, vdim)
     gate = sigmoid(h @ t[p + "g"].T)
