@@ -23,6 +23,14 @@ __device__ __forceinline__ float gelu_tanh_ratio(float z) {
   return z / (1.f + expf(-2.f * t));
 }
 
+__device__ __forceinline__ void store4(float* p, float a, float b, float c, float d) {
+  *reinterpret_cast<float4*>(p) = make_float4(a, b, c, d);
+}
+__device__ __forceinline__ void store4(__nv_bfloat16* p, float a, float b, float c, float d) {
+  __nv_bfloat162 v[2] = {__floats2bfloat162_rn(a, b), __floats2bfloat162_rn(c, d)};
+  *reinterpret_cast<uint2*>(p) = *reinterpret_cast<const uint2*>(v);
+}
+
 template <typename T>
 __global__ void cast_rows_kernel(const float* __restrict__ x, int ld_x, T* __restrict__ out,
                                  int ld_out, int rows, int width) {
@@ -60,6 +68,43 @@ __global__ void gated_unit_kernel(const float* __restrict__ gate, int ld_gate,
     }
     stf(out + (size_t)r * ld_out + c, a * b);
   }
+}
+
+// The unit of two fp32 matrices in pieces of four entries: a CTA's threads side by side along a
+// row, rows along grid.y (no division per entry), 16-byte loads. For rows that start on 16-byte
+// boundaries and are whole pieces.
+template <typename T, int ACT>
+__global__ void __launch_bounds__(256)
+gated_unit4_kernel(const float* __restrict__ gate, int ld_gate, const float* __restrict__ other,
+                   int ld_other, T* __restrict__ out, int ld_out, int rows, int width) {
+  pdl_launch_dependents();
+  pdl_wait_for(gate, other);
+  const int c = (blockIdx.x * blockDim.x + threadIdx.x) * 4;
+  if (c >= width) return;
+  for (int r = blockIdx.y; r < rows; r += gridDim.y) {
+    const float4 g = *reinterpret_cast<const float4*>(gate + (size_t)r * ld_gate + c);
+    const float4 b = *reinterpret_cast<const float4*>(other + (size_t)r * ld_other + c);
+    auto act = [](float z) {
+      return ACT == GATE_GELU_TANH ? gelu_tanh_ratio(z) : z / (1.f + expf(-z));
+    };
+    store4(out + (size_t)r * ld_out + c, act(g.x) * b.x, act(g.y) * b.y, act(g.z) * b.z,
+           act(g.w) * b.w);
+  }
+}
+
+template <typename T>
+int gated_unit4(const float* gate, int ld_gate, const float* other, int ld_other, int act, T* out,
+                int ld_out, int rows, int width, cudaStream_t s) {
+  const int pieces = width / 4, threads = pieces >= 256 ? 256 : (pieces + 31) / 32 * 32;
+  const int across = (pieces + threads - 1) / threads;
+  const int most = sm_count() * 16 / across + 1;  // rows of CTAs: about sixteen CTAs an SM
+  const dim3 grid(across, rows < most ? rows : most);
+  if (act == GATE_GELU_TANH) {
+    return launch_kernel(gated_unit4_kernel<T, GATE_GELU_TANH>, grid, dim3(threads), 0, s, 1, gate,
+                         ld_gate, other, ld_other, out, ld_out, rows, width);
+  }
+  return launch_kernel(gated_unit4_kernel<T, GATE_SILU>, grid, dim3(threads), 0, s, 1, gate,
+                       ld_gate, other, ld_other, out, ld_out, rows, width);
 }
 
 enum UnaryAct : int { UNARY_TANH = 0, UNARY_XIELU = 1 };
@@ -145,6 +190,16 @@ AYK_API int ayk_gated_unit(const float* gate, int ld_gate, const float* other, i
   }
   const int threads = 256, blocks = blocks_for((long long)rows * width, threads);
   cudaStream_t s = (cudaStream_t)stream;
+  if (other != nullptr && width % 4 == 0 && ld_gate % 4 == 0 && ld_other % 4 == 0 &&
+      ld_out % 4 == 0 && (uintptr_t)gate % 16 == 0 && (uintptr_t)other % 16 == 0 &&
+      (uintptr_t)out % 16 == 0 && (type == 0 || type == 1)) {
+    if (type == 0) {
+      return gated_unit4<float>(gate, ld_gate, other, ld_other, act, (float*)out, ld_out, rows,
+                                width, s);
+    }
+    return gated_unit4<__nv_bfloat16>(gate, ld_gate, other, ld_other, act, (__nv_bfloat16*)out,
+                                      ld_out, rows, width, s);
+  }
   if (type == 0) {
     return launch_kernel(gated_unit_kernel<float, float>, dim3(blocks), dim3(threads), 0, s, 1,
                          gate, ld_gate, other, ld_other, (const float*)table, ld_table, index,

@@ -366,3 +366,23 @@ def test_the_norm_of_two_scaled_branches(width, dtype):
     assert torch.equal(copy[:rows], got[:rows].to(dtype)) and float(copy[rows].abs().max()) == 0.0
     with pytest.raises(BackendError):
         ops.norm_add(x.to(DEV), w.to(DEV), eps, got, rows=rows, x_factor=0.6)
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("activation", ["silu", "gelu_tanh"])
+@pytest.mark.parametrize("rows,width", [(1, 4), (9, 21), (3, 1028), (700, 36), (2500, 8)])
+def test_gated_units_of_whole_and_broken_pieces(dtype, activation, rows, width):
+    """The two halves of one product's rows; entries beyond the unit stay as they were."""
+    both = randn(rows, 2 * width, seed=1, scale=2.0).float()
+    out = torch.full((rows + 1, width + (4 if width % 4 == 0 else 3)), 7.0, dtype=dtype, device=DEV)
+    halves = both.to(DEV)
+    ops.gated_unit(halves[:, :width], out[:, :width], activation=activation, rows=rows,
+                   other=halves[:, width:])
+    g, b = both[:, :width].double(), both[:, width:].double()
+    if activation == "silu":
+        want = g * torch.sigmoid(g) * b
+    else:
+        want = torch.nn.functional.gelu(g, approximate="tanh") * b
+    close(out[:rows, :width], want, 3e-6 if dtype == torch.float32 else 5e-3)
+    assert float((out[rows].float() - 7.0).abs().max()) == 0.0
+    assert float((out[:, width:].float() - 7.0).abs().max()) == 0.0
