@@ -103,6 +103,24 @@ __device__ __forceinline__ float activate_to_bf16(float x, int act) {
   return x;
 }
 
+// The activation of a tile's row piece. The choice is made once, around the loops: a test per
+// element makes the compiler branch in every step of an unrolled epilogue, which then takes longer
+// than the tile's main loop.
+template <bool TO_BF16, int N>
+__device__ __forceinline__ void activate_all(float (&v)[N], int act) {
+  if (act == ACT_NONE) return;
+  if (act == ACT_GELU_TANH) {
+#pragma unroll
+    for (int j = 0; j < N; ++j) v[j] = TO_BF16 ? gelu_tanh_fast(v[j]) : gelu_tanh(v[j]);
+  } else if (act == ACT_GELU_ERF) {
+#pragma unroll
+    for (int j = 0; j < N; ++j) v[j] = gelu_erf(v[j]);
+  } else {
+#pragma unroll
+    for (int j = 0; j < N; ++j) v[j] = relu_squared(v[j]);
+  }
+}
+
 // Programmatic dependent launch: a kernel launched with the attribute may start while its
 // predecessor in the stream is still running; pdl_wait() blocks until the predecessor has
 // finished and its writes are visible, so everything before it (barrier set-up, tensor-memory

@@ -141,22 +141,39 @@ __device__ __forceinline__ float dot_row(const float* q, const float* k, int dim
   return sum;
 }
 __device__ __forceinline__ float dot_row(const float* q, const __nv_bfloat16* k, int dim) {
-  float sum = 0.f;
+  float sum = 0.f, sum2 = 0.f;  // two chains
   if (dim % 8 == 0) {
-    for (int d = 0; d < dim; d += 8) {
+    // four pieces in flight at a time (a thread's row is its own: nobody else fetches ahead)
+    int d = 0;
+    for (; d + 32 <= dim; d += 32) {
+      uint4 raw[4];
+#pragma unroll
+      for (int u = 0; u < 4; ++u) raw[u] = *reinterpret_cast<const uint4*>(k + d + 8 * u);
+#pragma unroll
+      for (int u = 0; u < 4; ++u) {
+        const __nv_bfloat162* pair = reinterpret_cast<const __nv_bfloat162*>(&raw[u]);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const float2 v = __bfloat1622float2(pair[i]);
+          sum = fmaf(q[d + 8 * u + 2 * i], v.x, sum);
+          sum2 = fmaf(q[d + 8 * u + 2 * i + 1], v.y, sum2);
+        }
+      }
+    }
+    for (; d < dim; d += 8) {
       const uint4 raw = *reinterpret_cast<const uint4*>(k + d);
       const __nv_bfloat162* pair = reinterpret_cast<const __nv_bfloat162*>(&raw);
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
         const float2 v = __bfloat1622float2(pair[i]);
         sum = fmaf(q[d + 2 * i], v.x, sum);
-        sum = fmaf(q[d + 2 * i + 1], v.y, sum);
+        sum2 = fmaf(q[d + 2 * i + 1], v.y, sum2);
       }
     }
   } else {
     for (int d = 0; d < dim; ++d) sum = fmaf(q[d], __bfloat162float(k[d]), sum);
   }
-  return sum;
+  return sum + sum2;
 }
 
 // One CTA per (row, head). The visible keys, numbered 0 .. total - 1 (kept ones first), are
@@ -373,6 +390,7 @@ gated_decode_kernel(const T* __restrict__ q, int ld_q, const T* __restrict__ k_p
 #pragma unroll
     for (int i = 0; i < VEC; ++i) acc[i] *= alpha;
     if (group < groups) {
+#pragma unroll 4
       for (int jj = group; jj < n; jj += groups) {
         float v[VEC];
         Piece<T>::load(v_pages + base_s[jj] * vdim + column * VEC, v);

@@ -68,8 +68,7 @@ __device__ __forceinline__ void store_row_chunk(const uint32_t* raw, int m, int 
   const bool full_chunk = n + 32 <= N;
   if (mode == OUT_BF16) {
     __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(out) + (size_t)m * ldo + n;
-#pragma unroll
-    for (int j = 0; j < 32; ++j) v[j] = activate(v[j], act);
+    activate_all<false>(v, act);
     if (vec_ok && full_chunk) {
 #pragma unroll
       for (int j = 0; j < 32; j += 8) {
@@ -92,10 +91,7 @@ __device__ __forceinline__ void store_row_chunk(const uint32_t* raw, int m, int 
     }
   } else {
     float* dst = reinterpret_cast<float*>(out) + (size_t)m * ldo + n;
-    if (mode == OUT_F32) {
-#pragma unroll
-      for (int j = 0; j < 32; ++j) v[j] = activate(v[j], act);
-    }
+    if (mode == OUT_F32) activate_all<false>(v, act);
     if (vec_ok && full_chunk) {
 #pragma unroll
       for (int j = 0; j < 32; j += 4) {
@@ -221,11 +217,9 @@ __device__ __forceinline__ void epilogue_warp(uint32_t acc, int lane, int m_warp
     if (mode == OUT_BF16) {
       // (the tanh of a GELU through the special-function unit: with tanhf the epilogue of a
       // 128 x 256 tile took longer than its main loop)
-#pragma unroll
-      for (int j = 0; j < 32; ++j) v[j] = activate_to_bf16(v[j], act);
+      activate_all<true>(v, act);
     } else if (mode == OUT_F32) {
-#pragma unroll
-      for (int j = 0; j < 32; ++j) v[j] = activate(v[j], act);
+      activate_all<false>(v, act);
     }
     if (mode == OUT_BF16) {
       const int piece0 = (c & 1) * 4;

@@ -21,7 +21,8 @@ from senurax_cases import assert_close, channel, delta, dense, layer, numpy_stat
 
 __all__ = ["LOUD", "LOUD_WIDE", "NAME", "TINY_A", "TINY_B", "TINY_C", "TINY_D", "assert_close",
            "attention", "channel", "delta", "dense", "greedy_generate", "latent", "layer",
-           "make_model", "model", "parallel", "plain_logits", "rotation", "stretched", "write_model"]
+           "make_model", "model", "numpy_state", "parallel", "plain_logits", "rotation", "stretched",
+           "write_model"]
 
 NAME = "Kakilorn"
 
