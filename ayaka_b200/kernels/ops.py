@@ -1951,7 +1951,8 @@ def norm_add(x: torch.Tensor, weight: torch.Tensor, eps: float, dst: torch.Tenso
         typed = next_out
     status = library("rms_norm").ayk_norm_add_next(
         _ptr(x), c_int(x.stride(0)), c_float(x_factor), _ptr(other),
-        c_int(0 if other is None else other.stride(0)), c_float(other_factor), _ptr(weight), c_float(weight_offset), c_float(eps),
+        c_int(0 if other is None else other.stride(0)), c_float(other_factor), _ptr(weight),
+        c_float(weight_offset), c_float(eps),
         c_float(factor), _ptr(dst), c_int(dst.stride(0)), _ptr(copy),
         c_int(0 if copy is None else copy.stride(0)),
         c_int(0 if typed is None else _TYPE[typed.dtype]),
@@ -1976,9 +1977,9 @@ def gated_attention_prepare(proj: torch.Tensor, *, k_offset: int, v_offset: int,
     dim`` keys at ``k_offset``, ``kv_heads * vdim`` values at ``v_offset``): queries and keys
     each normalised by the root mean square over their whole projection with a weight per
     entry (``None``: no norm), or with ``head_norm`` every head by its own root mean square with
-    one weight of ``dim`` entries for all heads, the first ``2 * len(freq)`` entries of every head rotated by the
-    row's position (``freq`` ``None``: no rotation; see :func:`rope`), the queries written to ``q`` ``[N, heads * dim]``, the key and
-    value into the row's cache slot (``k_pages`` ``[page, kv_head, slot, dim]``, ``v_pages``
+    one weight of ``dim`` entries for all heads, the first ``2 * len(freq)`` entries of
+    every head rotated by the row's position (``freq`` ``None``: no rotation; see :func:`rope`), the
+    queries written to ``q`` ``[N, heads * dim]``, the key and value into the row's cache slot (``k_pages`` ``[page, kv_head, slot, dim]``, ``v_pages``
     likewise with ``vdim``; ``None``: stored nowhere)."""
     op = "gated_attention_prepare"
     if _left_out and op in _left_out:
@@ -2057,8 +2058,8 @@ def gated_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tenso
     key/value head ``h // (heads / kv_heads)``; scores ``scale * q . k``, with ``slope`` (float32
     ``[heads]``) less ``slope[h] * (p - j)``; weights in fp32: ``scores="softmax"`` over the
     visible keys, or ``scores="sigmoid"``: each visible key's own ``sigmoid(score +
-    score_bias[h])`` (``score_bias`` float32 ``[heads]``, optional); with ``gate`` (float32 ``[N, heads * vdim]``) the result is multiplied entry by
-    entry by ``sigmoid(gate)``. The step's own keys must already be stored."""
+    score_bias[h])`` (``score_bias`` float32 ``[heads]``, optional); with ``gate``
+    (float32 ``[N, heads * vdim]``) the result is multiplied entry by entry by ``sigmoid(gate)``. The step's own keys must already be stored."""
     op = "gated_attention"
     if _left_out and op in _left_out:
         return
