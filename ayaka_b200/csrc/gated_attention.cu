@@ -12,8 +12,9 @@
 // square (one mean over all heads' entries, eps inside the root) and multiplied by a weight
 // per entry, or, with head_norm, every head by its own root mean square and multiplied by one
 // weight of dim entries that all heads share; with rotation frequencies the first rot_dims entries
-// of every query and key head are then rotated by the row's position; queries go to `q` in the compute type, the key and
-// value into the row's cache slot (pages [page][kv head][slot][dim or vdim]).
+// of every query and key head are then rotated by the row's position; queries go to `q` in the
+// compute type, the key and value into the row's cache slot (pages [page][kv head][slot][dim or
+// vdim]).
 //
 // attention: scores scale * (q . k), weights and the weighted sum in fp32, the result times
 // sigmoid(gate) entry by entry when a gate (fp32, [row][H * vdim]) is given. With `slope` (fp32,

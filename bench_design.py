@@ -165,7 +165,7 @@ def kakilorn_config(width: int, heads: int, ff: int, repeats: int, vocab: int) -
               "q_rank": width // 2, "kv_rank": 256 - head // 2,
               "scale": (head + head // 2) ** -0.5,
               "rot": {"base": 500000.0, "dims": head // 2,
-                      "scaling": {"factor": 4.0, "original": 8192, "fast": 32.0, "slow": 1.0}}}
+                      "scaling": {"factor": 8.0, "original": 8192, "fast": 16.0, "slow": 1.0}}}
     delta = {"heads": width // 64, "kv_heads": width // 64, "dim": 64, "vdim": 64, "conv": 4}
     left = {"heads": heads, "kv_heads": heads // 4, "dim": head, "vdim": head,
             "scale": head ** -0.5,

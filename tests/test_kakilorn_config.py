@@ -172,7 +172,7 @@ def test_frequencies_and_slopes_are_the_plain_ones():
         assert np.allclose(distance_slopes(heads), plain.slopes(heads), rtol=1e-15)
     assert distance_slopes(8)[0] == 0.5 and distance_slopes(8)[7] == 2.0 ** -8
     for rot in (rotation(8, 50.0, stretched(4.0, 64, 8.0, 1.0)), rotation(6, 37.0),
-                rotation(32, 500000.0, stretched(3.0, 2048)),
+                rotation(24, 250000.0, stretched(3.0, 2048, 24.0)),
                 rotation(10, 9.0, stretched(2.0, 20, 5.0, 0.5))):
         want, want_gain = plain.rotary_frequencies(rot)
         got, gain = blended_frequencies(rot["dims"], rot["base"], **(rot.get("scaling") or {}))

@@ -82,7 +82,7 @@ CASES = [
     (4, 2, 16, 8, 9, 13, 8),
     (3, 1, 8, 20, 1, 0, 16),
     (2, 2, 12, 8, 0, 0, 16),
-    (8, 1, 96, 96, 70, 21, 16),
+    (7, 1, 72, 104, 70, 21, 16),
     (5, 5, 24, 40, 33, 1, 32),
 ]
 
@@ -134,7 +134,7 @@ def test_weights_that_fall_with_the_distance(dtype, scores, sloped, biased, case
 
 
 TILED = [
-    (8, 1, 96, 96, 136, 20, 16),
+    (6, 1, 80, 112, 150, 30, 16),
     (4, 2, 48, 80, 130, 70, 16),   # kept keys beyond one tile of keys
     (2, 2, 16, 32, 64, 64, 8),     # the window and the kept stretch end on a tile's edge
     (3, 1, 64, 64, 0, 9, 16),      # no window: nothing is kept apart
@@ -280,7 +280,7 @@ def test_latent_prepare_with_blended_frequencies_and_their_gain(dtype):
 
 @pytest.mark.parametrize("kernel", ["generic", "single", "flash"])
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("heads,rank,rot,page", [(3, 24, 8, 16), (6, 128, 32, 16), (18, 96, 0, 8),
+@pytest.mark.parametrize("heads,rank,rot,page", [(3, 24, 8, 16), (5, 112, 48, 16), (18, 96, 0, 8),
                                                  (2, 40, 24, 32)])
 def test_the_sink_of_latent_attention(kernel, dtype, heads, rank, rot, page):
     """Sinks from far below the scores (no effect) to far above (the head says nothing)."""
